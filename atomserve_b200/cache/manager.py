@@ -12,7 +12,7 @@ can meet a NaN (atomserve/kv_cache.py:112-118).
 Pages come back when a request ends or is preempted, and, in a group with a window or with
 chunks, as soon as no later position can read them: before a step that starts at position c,
 pages wholly below c - window + 1 (below the start of c's chunk) are released and their table
-entries set to -1.
+entries set to -1; where the first positions stay visible (`PageSpec.keep_first`), their pages stay.
 
 The reference has one uniform pool (atomserve/kv_cache.py:89-135) and lets the scheduler talk to
 the allocator directly (atomserve/scheduler.py:204-254); here the scheduler talks to this
@@ -147,17 +147,21 @@ class CacheManager:
         """The lowest logical page a step starting at position `start` can still read."""
         return group.spec.first_needed(start) // self.block_size
 
+    def kept_blocks(self, group: CacheGroup) -> int:
+        """How many of a request's first pages hold positions that every later one reads."""
+        return -(-group.spec.keep_first // self.block_size)
+
     def release_passed(self, rc: RequestCache, start: int) -> None:
         """Give back the pages that no position from `start` on can read (a window has passed them, or
         they lie before the chunk that `start` is in)."""
         for g, table in zip(self.groups, rc.block_tables):
             if not g.releases_early:
                 continue
-            upto = min(self.first_needed_block(g, start), len(table))
-            passed = [b for b in table[:upto] if b >= 0]
+            upto, kept = min(self.first_needed_block(g, start), len(table)), self.kept_blocks(g)
+            passed = [b for b in table[kept:upto] if b >= 0]
             if passed:
                 g.allocator.free(passed)
-                for i in range(upto):
+                for i in range(kept, upto):
                     table[i] = -1
 
     def reserve(self, rc: RequestCache, start: int, num_new: int) -> bool:

@@ -19,6 +19,14 @@
 // computed for a row does not depend on what else is in the batch. With one partition the block
 // writes the output; otherwise it writes (max, sum, accumulator) and `attention_reduce` merges.
 //
+// Heads of several key parts (`parts` > 1): a query row holds one vector per key head and its score
+// is the sum of their products, sum over c of q[row, c] . k[c], so every query head reads the keys
+// of all kv heads (its values still come from kv head h / G). That is how scores that are mixed
+// across heads run: the mix moves into the queries.
+//
+// Kept first positions (`keep`): positions below it stay visible whatever the window or chunk says.
+// The block of a row's first partition visits them before its own keys.
+//
 // Keys are visited in tiles of 32 at absolute multiples of 32; lane = key for the scores, lane =
 // output column (mod 32) for the weighted sum of values.
 #include "common.cuh"
@@ -31,7 +39,7 @@ constexpr int kMaxRows = kWarps * kRowsPerWarp;  // 32
 constexpr int kKeyTile = 32;
 
 struct AttentionParams {
-  const void* q;         // [T, H, hd]
+  const void* q;         // [T, H, parts, hd]
   void* out;             // [T, H, hd]
   const void* k_cache;   // [num_blocks, KV, bs, hd]
   const void* v_cache;
@@ -49,6 +57,8 @@ struct AttentionParams {
   int chunk;                 // 0: none; else a query sees only the keys of its own run of `chunk`
                              // positions (runs counted from position 0 of the request)
   float softcap;             // 0: none; else score <- softcap tanh(score / softcap)
+  int keep;                  // positions below it are seen from everywhere behind them
+  int parts;                 // 1: a query head reads its own kv head's keys; KV: those of all kv heads
   int PS, NP;                // partition size in keys, number of partitions (grid.z)
   float scale;
 };
@@ -94,13 +104,18 @@ paged_attention_kernel(const AttentionParams p) {
   const int part = lo / p.PS + blockIdx.z;
   const int key_lo = max(lo, part * p.PS);
   const int key_hi = (int)min((long long)hi, (long long)(part + 1) * p.PS);
+  // kept positions that lie before the first key of the block's rows: the first partition's
+  const int kept = blockIdx.z == 0 ? min(p.keep, lo) : 0;
 
   const T* q = (const T*)p.q;
-  for (int i = threadIdx.x; i < num_rows * hd; i += blockDim.x) {
-    const int rr = i / hd, e = i - rr * hd;
-    const int qi = rr / gc, g = rr - qi * gc;
-    q_s[rr * hd + e] = asb::to_float(q[((size_t)(row0 + qi) * p.H + head0 + g) * hd + e]) * p.scale;
-  }
+  auto load_queries = [&](int c) {
+    for (int i = threadIdx.x; i < num_rows * hd; i += blockDim.x) {
+      const int rr = i / hd, e = i - rr * hd;
+      const int qi = rr / gc, g = rr - qi * gc;
+      q_s[rr * hd + e] = asb::to_float(q[(((size_t)(row0 + qi) * p.H + head0 + g) * p.parts + c) * hd + e]) * p.scale;
+    }
+  };
+  if (p.parts == 1) load_queries(0);
 
   float m[kRowsPerWarp], l[kRowsPerWarp], acc[kRowsPerWarp][EPL];
 #pragma unroll
@@ -115,26 +130,43 @@ paged_attention_kernel(const AttentionParams p) {
   const T* vc = (const T*)p.v_cache;
   const int* table = p.block_tables + (size_t)r * p.table_width;
 
-  for (int kt0 = (key_lo / kKeyTile) * kKeyTile; kt0 < key_hi; kt0 += kKeyTile) {
+  const int main_begin = (key_lo / kKeyTile) * kKeyTile;
+  const int kept_end = min((kept + kKeyTile - 1) / kKeyTile * kKeyTile, main_begin);  // tiles that hold nothing but kept positions
+  for (int kt0 = kept_end > 0 ? 0 : main_begin; kt0 < key_hi; kt0 = kt0 + kKeyTile == kept_end ? main_begin : kt0 + kKeyTile) {
     __syncthreads();  // previous tile fully consumed (and q_s written, first time round)
     if (threadIdx.x < kKeyTile) {
       const int j = kt0 + threadIdx.x;
-      block_of_key[threadIdx.x] = (j >= key_lo && j < key_hi) ? table[j / p.bs] : -1;
+      block_of_key[threadIdx.x] = ((j >= key_lo && j < key_hi) || j < kept) ? table[j / p.bs] : -1;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < kKeyTile * hd; i += blockDim.x) {
-      const int jj = i / hd, e = i - jj * hd;
-      const int blk = block_of_key[jj];
-      float kv = 0.f, vv = 0.f;
-      if (blk >= 0) {
-        const size_t at = (((size_t)blk * p.KV + kvh) * p.bs + (kt0 + jj) % p.bs) * hd + e;
-        kv = asb::to_float(kc[at]);
-        vv = asb::to_float(vc[at]);
+    float d[kRowsPerWarp];
+#pragma unroll
+    for (int s = 0; s < kRowsPerWarp; ++s) d[s] = 0.f;
+    for (int c = 0; c < p.parts; ++c) {
+      if (c > 0) __syncthreads();  // the part before has been read
+      if (p.parts > 1) load_queries(c);
+      const int key_head = p.parts > 1 ? c : kvh;
+      for (int i = threadIdx.x; i < kKeyTile * hd; i += blockDim.x) {
+        const int jj = i / hd, e = i - jj * hd;
+        const int blk = block_of_key[jj];
+        float kv = 0.f;
+        const size_t in_page = (size_t)((kt0 + jj) % p.bs) * hd + e;
+        if (blk >= 0) kv = asb::to_float(kc[((size_t)blk * p.KV + key_head) * p.bs * hd + in_page]);
+        k_s[jj * kstride + e] = kv;
+        if (c == 0) v_s[jj * hd + e] = blk >= 0 ? asb::to_float(vc[((size_t)blk * p.KV + kvh) * p.bs * hd + in_page]) : 0.f;
       }
-      k_s[jj * kstride + e] = kv;
-      v_s[jj * hd + e] = vv;
+      __syncthreads();
+#pragma unroll
+      for (int s = 0; s < kRowsPerWarp; ++s) {
+        const int rr = warp + s * kWarps;
+        if (rr >= num_rows) break;
+        const float* qrow = q_s + rr * hd;
+        const float* krow = k_s + lane * kstride;
+        float a = d[s];
+        for (int e = 0; e < hd; ++e) a = fmaf(qrow[e], krow[e], a);
+        d[s] = a;
+      }
     }
-    __syncthreads();
 
     const int j = kt0 + lane;
     const bool in_range = block_of_key[lane] >= 0;
@@ -143,16 +175,9 @@ paged_attention_kernel(const AttentionParams p) {
       const int rr = warp + s * kWarps;
       if (rr >= num_rows) break;
       const int pq = pos0 + rr / gc;
-      const bool visible = in_range && j <= pq && (p.window <= 0 || j > pq - p.window) &&
-                           (p.chunk <= 0 || j >= pq - pq % p.chunk);
-      float score = -INFINITY;
-      if (visible) {
-        const float* qrow = q_s + rr * hd;
-        const float* krow = k_s + lane * kstride;
-        float d = 0.f;
-        for (int e = 0; e < hd; ++e) d = fmaf(qrow[e], krow[e], d);
-        score = p.softcap > 0.f ? p.softcap * tanhf(d / p.softcap) : d;
-      }
+      const bool visible = in_range && j <= pq &&
+                           (((p.window <= 0 || j > pq - p.window) && (p.chunk <= 0 || j >= pq - pq % p.chunk)) || j < p.keep);
+      const float score = visible ? (p.softcap > 0.f ? p.softcap * tanhf(d[s] / p.softcap) : d[s]) : -INFINITY;
       const float m_new = fmaxf(m[s], asb::warp_max(score));
       if (m_new == -INFINITY) continue;  // this row sees none of these keys
       const float corr = expf(m[s] - m_new);
@@ -364,15 +389,16 @@ extern "C" void asb_attention_tile_shape(int G, int* QT, int* GC) {
 
 // Float scratch needed when NP > 1: part_m and part_l take T*H*NP floats each, part_acc
 // T*H*NP*hd. Every partition slot of every row is written before the reduction reads it.
-// `chunk` and `softcap` (0: none): see AttentionParams.
-extern "C" int asb_paged_attention_masked(void* out, const void* q, const void* k_cache,
+// `chunk`, `softcap`, `keep` (0: none) and `parts` (1 or KV; q is [T, H, parts, hd]): see AttentionParams.
+extern "C" int asb_paged_attention_parts(void* out, const void* q, const void* k_cache,
                                           const void* v_cache, const int* block_tables,
                                           const int* req_q_start, const int* req_pos_start,
                                           float* part_m, float* part_l, float* part_acc, const float* sink,
                                           int num_tokens, int R, int H, int KV, int hd, int bs,
-                                          int table_width, int window, int chunk, int PS, int NP, float scale,
-                                          float softcap, int dtype, cudaStream_t stream) {
+                                          int table_width, int window, int chunk, int keep, int parts, int PS, int NP,
+                                          float scale, float softcap, int dtype, cudaStream_t stream) {
   if (num_tokens == 0 || R == 0) return 0;
+  if (keep < 0 || (parts != 1 && parts != KV)) return asb::fail("paged_attention: keep %d must not be negative, parts %d must be 1 or %d", keep, parts, KV);
   if (KV < 1 || H % KV) return asb::fail("paged_attention: %d heads over %d kv heads", H, KV);
   if (hd < 1 || hd > 256) return asb::fail("paged_attention: head_dim %d not in 1..256", hd);
   if (NP < 1 || PS < kKeyTile || PS % kKeyTile) return asb::fail("paged_attention: partition size %d must be a positive multiple of %d", PS, kKeyTile);
@@ -387,9 +413,21 @@ extern "C" int asb_paged_attention_masked(void* out, const void* q, const void* 
   p.HC = (H / KV + p.GC - 1) / p.GC;
   if (p.KV * p.HC > 65535) return asb::fail("paged_attention: too many head chunks");
   if (chunk < 0 || softcap < 0.f) return asb::fail("paged_attention: chunk %d and softcap %f must not be negative", chunk, (double)softcap);
-  p.window = window; p.chunk = chunk; p.softcap = softcap; p.PS = PS; p.NP = NP; p.scale = scale;
+  p.window = window; p.chunk = chunk; p.softcap = softcap; p.keep = keep; p.parts = parts; p.PS = PS; p.NP = NP; p.scale = scale;
   ASB_DISPATCH_DTYPE(dtype, T, return launch<T>(p, num_tokens, stream));
   return 0;
+}
+
+extern "C" int asb_paged_attention_masked(void* out, const void* q, const void* k_cache,
+                                          const void* v_cache, const int* block_tables,
+                                          const int* req_q_start, const int* req_pos_start,
+                                          float* part_m, float* part_l, float* part_acc, const float* sink,
+                                          int num_tokens, int R, int H, int KV, int hd, int bs,
+                                          int table_width, int window, int chunk, int PS, int NP, float scale,
+                                          float softcap, int dtype, cudaStream_t stream) {
+  return asb_paged_attention_parts(out, q, k_cache, v_cache, block_tables, req_q_start, req_pos_start, part_m, part_l,
+                                   part_acc, sink, num_tokens, R, H, KV, hd, bs, table_width, window, chunk, 0, 1, PS, NP,
+                                   scale, softcap, dtype, stream);
 }
 
 extern "C" int asb_paged_attention_sink(void* out, const void* q, const void* k_cache,

@@ -6,13 +6,16 @@
 //                     groups of neighbouring experts, a group's score is the sum of its `group_top`
 //                     largest scores and only experts of the `keep` best groups can be chosen. The
 //                     `top` largest allowed scores win (ties: the lower index); their weights are
-//                     s / (sum s + 1e-20) * scale (`renorm` 0: s * scale). Column `gate_col` of z,
+//                     s / (sum s + 1e-20) * scale (`renorm` 0: s * scale). `softmax` 2: the `top`
+//                     largest of z + bias are chosen and weighted by the softmax over the chosen
+//                     alone, times scale. Column `gate_col` of z,
 //                     if not negative, gives sigmoid(z) per token: the gate of a shared expert.
 //   asb_moe_group     pairs sorted by expert: offsets [E + 1], the token of each sorted row, and
 //                     for each (token, choice) its sorted row
 //   asb_moe_glu       hidden[row] = act(x[token] . gate_e^T, x[token] . up_e^T) for the rows of
 //                     each expert e: g = min(., limit), u = clamp(., -limit, limit),
 //                     g sigmoid(slope g) (u + shift); limit <= 0: no clamping
+//   asb_moe_relu2     hidden[row] = max(x[token] . up_e^T, 0)^2: experts without a gate
 //   asb_moe_down      y[row] = hidden[row] . down_e^T, float32
 //   asb_moe_combine   out[t] = sum_k weight[t, k] y[row(t, k)] (+ shared_gate[t] * shared[t]), float32,
 //                     the choices added in their order of selection
@@ -35,6 +38,7 @@ struct RouteParams {
   float* weights;  // [T, top]
   float* shared_gate;  // [T] or null
   const float* bias;   // [E] or null: added to the scores for the final choice only, not to the weights
+                       // (softmax 2: part of the logits)
 };
 
 // one warp per token; scores and masks in shared memory
@@ -47,7 +51,7 @@ __global__ void moe_route_kernel(const RouteParams p) {
   float* gs = allowed + p.E;     // [G] group scores
   const int t = blockIdx.x, lane = threadIdx.x;
   const float* z = p.z + (size_t)t * p.stride;
-  if (p.softmax) {
+  if (p.softmax == 1) {
     float mx = -INFINITY;
     for (int e = lane; e < p.E; e += 32) mx = fmaxf(mx, z[e]);
     mx = asb::warp_max(mx);
@@ -55,6 +59,8 @@ __global__ void moe_route_kernel(const RouteParams p) {
     for (int e = lane; e < p.E; e += 32) sum += expf(z[e] - mx);
     sum = asb::warp_sum(sum);
     for (int e = lane; e < p.E; e += 32) s[e] = expf(z[e] - mx) / sum;
+  } else if (p.softmax == 2) {
+    for (int e = lane; e < p.E; e += 32) s[e] = p.bias ? z[e] + p.bias[e] : z[e];
   } else {
     for (int e = lane; e < p.E; e += 32) s[e] = 1.f / (1.f + expf(-z[e]));
   }
@@ -100,13 +106,14 @@ __global__ void moe_route_kernel(const RouteParams p) {
     }
   }
   float sum = 0.f;
+  float first = 0.f;  // the largest chosen logit (softmax 2)
   float mine = 0.f;  // lane k keeps the k-th chosen score
   int mine_at = 0;
   for (int n = 0; n < p.top; ++n) {
     float best = -INFINITY;
     int at = 0x7fffffff;
     for (int e = lane; e < p.E; e += 32) {
-      const float c = p.bias ? s[e] + p.bias[e] : s[e];
+      const float c = p.bias && p.softmax != 2 ? s[e] + p.bias[e] : s[e];
       if (allowed[e] > 0.f && c > best) { best = c; at = e; }
     }
     for (int o = 16; o > 0; o >>= 1) {
@@ -120,6 +127,10 @@ __global__ void moe_route_kernel(const RouteParams p) {
       if (lane == 0) allowed[at] = 0.f;
     }
     __syncwarp();
+    if (p.softmax == 2) {  // relative to the largest, which is chosen first
+      if (n == 0) first = best;
+      best = expf(best - first);
+    }
     sum += best;
     if ((n & 31) == lane) {
       // (top <= 32 is checked on the host)
@@ -129,7 +140,7 @@ __global__ void moe_route_kernel(const RouteParams p) {
   }
   if (lane < p.top) {
     p.ids[(size_t)t * p.top + lane] = mine_at;
-    p.weights[(size_t)t * p.top + lane] = (p.renorm ? mine / (sum + 1e-20f) : mine) * p.scale;
+    p.weights[(size_t)t * p.top + lane] = (p.softmax == 2 ? mine / sum : p.renorm ? mine / (sum + 1e-20f) : mine) * p.scale;
   }
   if (p.shared_gate && p.gate_col >= 0 && lane == 0) p.shared_gate[t] = 1.f / (1.f + expf(-z[p.gate_col]));
 }
@@ -180,7 +191,8 @@ struct GroupedParams {
   float limit, slope, shift;
 };
 
-template <typename TIn, typename TOut, bool GLU>
+// RELU2: one matrix, gathered rows, max(., 0)^2 of the sums (GLU is then false)
+template <typename TIn, typename TOut, bool GLU, bool RELU2 = false>
 __global__ void __launch_bounds__(256)
 grouped_gemm_kernel(const GroupedParams p) {
   asb::pdl_wait();
@@ -202,7 +214,7 @@ grouped_gemm_kernel(const GroupedParams p) {
   const int m0 = tile * BM, n0 = blockIdx.x * BN;
   const int rows = min(BM, count - m0);
   const int tid = threadIdx.x;
-  if (tid < BM) src_row[tid] = tid < rows ? (GLU ? p.row_token[begin + m0 + tid] : begin + m0 + tid) : -1;
+  if (tid < BM) src_row[tid] = tid < rows ? (GLU || RELU2 ? p.row_token[begin + m0 + tid] : begin + m0 + tid) : -1;
   __syncthreads();
   const int tx = tid % 16, ty = tid / 16;
   const int lrow = tid / 4, lk = (tid % 4) * 4;
@@ -282,6 +294,10 @@ grouped_gemm_kernel(const GroupedParams p) {
         }
         v = g / (1.f + expf(-p.slope * g)) * (u + p.shift);
       }
+      if constexpr (RELU2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      }
       out[orow + n] = asb::from_float<TOut>(v);
     }
   }
@@ -323,6 +339,7 @@ extern "C" int asb_moe_route_biased(const float* z, int stride, int T, int E, in
                                     float* weights, float* shared_gate, cudaStream_t stream) {
   if (T == 0) return 0;
   if (E < 1 || top < 1 || top > 32 || top > E) return asb::fail("moe_route: top %d of %d experts (at most 32)", top, E);
+  if (softmax < 0 || softmax > 2 || (softmax == 2 && G != 1)) return asb::fail("moe_route: score kind %d with %d groups", softmax, G);
   if (G < 1 || E % G || keep < 1 || keep > G) return asb::fail("moe_route: %d experts in %d groups, %d kept", E, G, keep);
   if ((size_t)(2 * E + G) * 4 > 48 * 1024) return asb::fail("moe_route: %d experts are too many", E);
   RouteParams p;
@@ -359,6 +376,18 @@ extern "C" int asb_moe_glu(void* hidden, const void* x, const int* row_token, co
   if (grid.y > 65535) return asb::fail("moe_glu: %d rows exceed the grid", pairs);
   ASB_DISPATCH_DTYPE(dtype, T, asb::launch(grouped_gemm_kernel<T, T, true>, grid, 256, 0, stream, p));
   return asb::check_launch("moe_glu");
+}
+
+extern "C" int asb_moe_relu2(void* hidden, const void* x, const int* row_token, const int* offsets, const void* up,
+                             int pairs, int E, int F, int K, int dtype, cudaStream_t stream) {
+  if (pairs == 0) return 0;
+  GroupedParams p;
+  p.out = hidden; p.x = x; p.row_token = row_token; p.offsets = offsets; p.w = up; p.w2 = nullptr;
+  p.E = E; p.N = F; p.K = K; p.limit = 0.f; p.slope = 1.f; p.shift = 0.f;
+  dim3 grid((F + BN - 1) / BN, row_tiles(pairs, E));
+  if (grid.y > 65535) return asb::fail("moe_relu2: %d rows exceed the grid", pairs);
+  ASB_DISPATCH_DTYPE(dtype, T, asb::launch(grouped_gemm_kernel<T, T, false, true>, grid, 256, 0, stream, p));
+  return asb::check_launch("moe_relu2");
 }
 
 extern "C" int asb_moe_down(float* y, const void* hidden, const int* offsets, const void* down, int pairs, int E,

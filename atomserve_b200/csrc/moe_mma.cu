@@ -8,6 +8,7 @@
 // depend on which rows share its tile.
 //
 //   asb_moe_glu_mma    hidden[row] = act(x[token] . gate_e^T, x[token] . up_e^T)   (bfloat16)
+//   asb_moe_relu2_mma  hidden[row] = max(x[token] . up_e^T, 0)^2                  (bfloat16)
 //   asb_moe_down_mma   y[row] = hidden[row] . down_e^T                            (float32)
 //
 // K must be a multiple of 8 and the operands 16-byte aligned (16-byte loads); the callers send
@@ -50,8 +51,9 @@ __device__ __forceinline__ void copy16(void* dst, const void* src, bool real) {
 }
 
 // WM warps along the rows (2: tiles of 64 rows, 4 warps; 4: tiles of 128 rows, 8 warps), two along
-// the columns; a warp computes 32 x 32 (and the same of the up matrix with GLU).
-template <bool GLU, int WM>
+// the columns; a warp computes 32 x 32 (and the same of the up matrix with GLU). RELU2: one matrix,
+// gathered rows, max(., 0)^2 of the sums, bfloat16 (GLU is then false).
+template <bool GLU, int WM, bool RELU2 = false>
 __global__ void __launch_bounds__(WM * 64)
 grouped_gemm_mma_kernel(const GroupedParams p) {
   constexpr int BM = WM * 32, kThreads = WM * 64;
@@ -73,7 +75,7 @@ grouped_gemm_mma_kernel(const GroupedParams p) {
   const int m0 = tile * BM, n0 = blockIdx.x * BN;
   const int rows = min(BM, count - m0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  if (tid < BM) src_row[tid] = tid < rows ? (GLU ? p.row_token[begin + m0 + tid] : begin + m0 + tid) : -1;
+  if (tid < BM) src_row[tid] = tid < rows ? (GLU || RELU2 ? p.row_token[begin + m0 + tid] : begin + m0 + tid) : -1;
   __syncthreads();
   const int K = p.K, N = p.N;
   const __nv_bfloat16* w = p.w + (size_t)e * N * K;
@@ -167,6 +169,9 @@ grouped_gemm_mma_kernel(const GroupedParams p) {
               up = fminf(fmaxf(up, -p.limit), p.limit);
             }
             ((__nv_bfloat16*)p.out)[orow + n] = __float2bfloat16_rn(gate / (1.f + expf(-p.slope * gate)) * (up + p.shift));
+          } else if constexpr (RELU2) {
+            const float r = fmaxf(v, 0.f);
+            ((__nv_bfloat16*)p.out)[orow + n] = __float2bfloat16_rn(r * r);
           } else {
             ((float*)p.out)[orow + n] = v;
           }
@@ -203,6 +208,22 @@ extern "C" int asb_moe_glu_mma(void* hidden, const void* x, const int* row_token
   if (big) asb::launch(grouped_gemm_mma_kernel<true, 4>, grid, 256, 0, stream, p);
   else asb::launch(grouped_gemm_mma_kernel<true, 2>, grid, 128, 0, stream, p);
   return asb::check_launch("moe_glu_mma");
+}
+
+extern "C" int asb_moe_relu2_mma(void* hidden, const void* x, const int* row_token, const int* offsets, const void* up,
+                                 int pairs, int E, int F, int K, cudaStream_t stream) {
+  if (pairs == 0) return 0;
+  if (!asb_moe_mma_supported(K) || !aligned16(x, up, nullptr)) return asb::fail("moe_relu2_mma: K = %d must be a multiple of 8 and the operands 16-byte aligned", K);
+  GroupedParams p;
+  p.out = hidden; p.x = (const __nv_bfloat16*)x; p.row_token = row_token; p.offsets = offsets;
+  p.w = (const __nv_bfloat16*)up; p.w2 = nullptr;
+  p.E = E; p.N = F; p.K = K; p.limit = 0.f; p.slope = 1.f; p.shift = 0.f;
+  const bool big = tall(pairs, E);
+  dim3 grid((F + BN - 1) / BN, row_tiles(pairs, E, big ? 128 : 64));
+  if (grid.y > 65535) return asb::fail("moe_relu2_mma: %d rows exceed the grid", pairs);
+  if (big) asb::launch(grouped_gemm_mma_kernel<false, 4, true>, grid, 256, 0, stream, p);
+  else asb::launch(grouped_gemm_mma_kernel<false, 2, true>, grid, 128, 0, stream, p);
+  return asb::check_launch("moe_relu2_mma");
 }
 
 extern "C" int asb_moe_down_mma(float* y, const void* hidden, const int* offsets, const void* down, int pairs, int E,

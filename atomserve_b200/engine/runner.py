@@ -175,7 +175,8 @@ class ModelRunner:
                     raise ValueError(f"block table holds {len(table) * bs} slots, the row needs {r.start + n}")
                 if g.releases_early:  # only windows and chunks release pages before a request ends
                     first = self.cache.first_needed_block(g, r.start)
-                    if any(b < 0 for b in table[first : -(-(r.start + n) // bs)]):
+                    kept = min(self.cache.kept_blocks(g), first)
+                    if any(b < 0 for b in table[first : -(-(r.start + n) // bs)]) or any(b < 0 for b in table[:kept]):
                         raise ValueError("a page the row still reads has been released")
 
     def _table_array(self, rc: RequestCache, g: int) -> np.ndarray:

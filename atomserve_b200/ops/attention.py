@@ -112,6 +112,7 @@ def paged_attention(
     sink: torch.Tensor | None = None,
     chunk: int | None = None,
     softcap: float | None = None,
+    keep_first: int = 0,
 ) -> torch.Tensor:
     """softmax(q k^T * scale) v for every new token, keys read in place from the pages.
 
@@ -127,14 +128,24 @@ def paged_attention(
     query sees only the keys of its own run (still j <= p). `softcap`: every scaled score becomes
     softcap * tanh(score / softcap) before the softmax (the sink is not capped).
 
+    `keep_first`: the first positions of a sequence, which stay visible behind the window and outside
+    the chunk. q may be [T, H, KV, hd], a vector per key head: a head's score is then the sum of the
+    products with all kv heads' keys (its values are still those of its own kv head): how scores that
+    are mixed across heads run, the mix being part of the queries.
+
     bfloat16 with head size 64 or 128 runs the tensor-core kernels (decode kernel for requests
     that bring at most 8 tokens, prefill kernel for longer portions; `host_q_lens`, the tokens
     each request brings, tells which are needed); everything else, and `generic=True`, runs the
     general CUDA-core kernel.
     """
     require_cuda(q, k_cache, v_cache, block_tables, req_q_start, req_pos_start)
-    T, H, hd = q.shape
     KV, bs = k_cache.shape[1], k_cache.shape[2]
+    parts = 1
+    if q.dim() == 4:
+        parts = q.shape[2]
+        if parts != KV:
+            raise KernelLibraryError(f"paged_attention: queries of {parts} parts against {KV} key heads")
+    T, H, hd = q.shape[0], q.shape[1], q.shape[-1]
     if not q.is_contiguous() or k_cache.shape != v_cache.shape or k_cache.shape[3] != hd:
         raise KernelLibraryError("paged_attention: q must be contiguous and the caches [blocks, KV, bs, hd]")
     if k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
@@ -144,13 +155,14 @@ def paged_attention(
             raise KernelLibraryError("paged_attention: index tensors must be contiguous int32")
     win = int(window) if window else 0
     chunk, softcap = int(chunk or 0), float(softcap or 0.0)
-    out = torch.empty_like(q)
+    out = torch.empty(T, H, hd, device=q.device, dtype=q.dtype)
     if sink is not None:
         require_cuda(sink)
         if sink.dtype != torch.float32 or sink.shape != (H,) or not sink.is_contiguous():
             raise KernelLibraryError(f"paged_attention: sink must be contiguous float32 [{H}]")
     span = min(win, chunk) if win and chunk else (win or chunk)  # a chunk bounds the keys of a row as a window does
-    if q.dtype == torch.bfloat16 and not generic and lib().asb_attention_mma_supported(hd, H // KV):
+    keep = int(keep_first) if span else 0
+    if q.dtype == torch.bfloat16 and not generic and parts == 1 and not keep and lib().asb_attention_mma_supported(hd, H // KV):
         return _paged_attention_mma(q, out, k_cache, v_cache, block_tables, req_q_start, req_pos_start,
                                     num_requests, max_context, win, scale, partitions, host_q_lens, sink, chunk, softcap, span)  # fmt: skip
     ps, np_ = partitions or plan_partitions(T, num_requests, KV, H // KV, max_context, span)
@@ -159,10 +171,10 @@ def paged_attention(
         part_m = torch.empty(T * H * np_, device=q.device, dtype=torch.float32)
         part_l = torch.empty_like(part_m)
         part_acc = torch.empty(T * H * np_ * hd, device=q.device, dtype=torch.float32)
-    check(lib().asb_paged_attention_masked(
+    check(lib().asb_paged_attention_parts(
         ptr(out), ptr(q), ptr(k_cache), ptr(v_cache), ptr(block_tables), ptr(req_q_start),
         ptr(req_pos_start), ptr(part_m), ptr(part_l), ptr(part_acc), ptr(sink), T, num_requests, H, KV, hd, bs,
-        block_tables.shape[1], win, chunk, ps, np_, float(scale), softcap, dtype_code(q), stream()))  # fmt: skip
+        block_tables.shape[1], win, chunk, keep, parts, ps, np_, float(scale), softcap, dtype_code(q), stream()))  # fmt: skip
     return out
 
 

@@ -4,6 +4,7 @@ sum back per token."""
 
 from __future__ import annotations
 
+import dataclasses
 import os
 
 import torch
@@ -22,11 +23,12 @@ def _tensor_cores(x: torch.Tensor, *weights: torch.Tensor) -> bool:
 
 
 def route(z: torch.Tensor, *, experts: int, top: int, groups: int = 1, group_top: int = 2, keep: int = 1,
-          scale: float = 1.0, gate_col: int | None = None, softmax: bool = False,
+          scale: float = 1.0, gate_col: int | None = None, softmax: bool | str = False,
           renormalise: bool = True, bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor | None]:  # fmt: skip
     """z: float32 [T, >= experts] router logits. Returns (ids int32 [T, top], weights float32
     [T, top], sigmoid(z[:, gate_col]) float32 [T] or None). `bias` (float32 [experts]) is added to
-    the scores for the final choice only; the weights are made of the scores themselves."""
+    the scores for the final choice only; the weights are made of the scores themselves.
+    `softmax="chosen"`: the `top` largest of z + bias, weighted by the softmax over those alone."""
     require_cuda(z, bias)
     if bias is not None and (bias.dtype != torch.float32 or bias.shape != (experts,) or not bias.is_contiguous()):
         raise KernelLibraryError(f"route: bias must be contiguous float32 [{experts}]")
@@ -37,7 +39,7 @@ def route(z: torch.Tensor, *, experts: int, top: int, groups: int = 1, group_top
     weights = torch.empty(T, top, device=z.device, dtype=torch.float32)
     shared = torch.empty(T, device=z.device, dtype=torch.float32) if gate_col is not None else None
     check(lib().asb_moe_route_biased(ptr(z), z.stride(0), T, experts, groups, group_top, keep, top,
-                                     -1 if gate_col is None else gate_col, int(softmax), int(renormalise), float(scale),
+                                     -1 if gate_col is None else gate_col, 2 if softmax == "chosen" else int(softmax), int(renormalise), float(scale),
                                      ptr(bias), ptr(ids), ptr(weights), ptr(shared), stream()))  # fmt: skip
     return ids, weights, shared
 
@@ -70,6 +72,32 @@ def experts_glu(x: torch.Tensor, row_token: torch.Tensor, offsets: torch.Tensor,
     check(lib().asb_moe_glu(ptr(hidden), ptr(x), ptr(row_token), ptr(offsets), ptr(gate), ptr(up), pairs, E, F, K,
                             float(limit), float(slope), float(shift), dtype_code(x), stream()))  # fmt: skip
     return hidden
+
+
+def experts_relu2(x: torch.Tensor, row_token: torch.Tensor, offsets: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """hidden [pairs, F]: for the sorted rows of expert e, max(x[token] . up[e]^T, 0)^2."""
+    require_cuda(x, row_token, offsets, up)
+    E, F, K = up.shape
+    if x.shape[1] != K or x.dtype != up.dtype or not (x.is_contiguous() and up.is_contiguous()):
+        raise KernelLibraryError("experts_relu2: x [T, K] against up [E, F, K] of one dtype, contiguous")
+    pairs = row_token.shape[0]
+    hidden = torch.empty(pairs, F, device=x.device, dtype=x.dtype)
+    if _tensor_cores(x, up):
+        check(lib().asb_moe_relu2_mma(ptr(hidden), ptr(x), ptr(row_token), ptr(offsets), ptr(up), pairs, E, F, K, stream()))
+        return hidden
+    check(lib().asb_moe_relu2(ptr(hidden), ptr(x), ptr(row_token), ptr(offsets), ptr(up), pairs, E, F, K, dtype_code(x), stream()))
+    return hidden
+
+
+@dataclasses.dataclass(frozen=True)
+class ExpertSums:
+    """What the experts gave, before the weighted sum back per token: the sorted rows' outputs
+    (float32 [pairs, width]) with each token's rows and weights [tokens, top]. A kernel that consumes
+    the sum can form it itself (`hyper_streams`); `combine` makes it a tensor."""
+
+    y: torch.Tensor
+    pair_row: torch.Tensor
+    weights: torch.Tensor
 
 
 def experts_down(hidden: torch.Tensor, offsets: torch.Tensor, down: torch.Tensor) -> torch.Tensor:

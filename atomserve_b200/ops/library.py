@@ -108,6 +108,12 @@ _SIGNATURES = {
     "asb_residual_dual_norm": [_P] * 9 + [_I, _I, _F, _F, _I, _P],
     "asb_pair_embedding": [_P] * 8 + [_I] * 8 + [_P, _P],
     "asb_concat_cast": [_P, _P, _P, _I, _I, _I, _P],
+    # parallel residual streams; scores mixed across heads, kept first positions; experts without a gate
+    "asb_hyper_streams": [_P] * 3 + [ctypes.c_longlong] * 2 + [_P, _I] + [_P] * 3 + [_I, _P] + [_I] * 5 + [_P] * 5 + [_I] * 3 + [_F, _I, _I, _P],
+    "asb_mixed_heads_prepare": [_P, _P] + [_I] * 5 + [_P] * 12 + [_I] * 10 + [_F, _F, _I, _P],
+    "asb_paged_attention_parts": [_P] * 11 + [_I] * 13 + [_F, _F, _I, _P],
+    "asb_moe_relu2": [_P] * 5 + [_I] * 5 + [_P],
+    "asb_moe_relu2_mma": [_P] * 5 + [_I] * 4 + [_P],
     # heads of several score maps
     "asb_qk_prepare_store": [_P] * 7 + [_I] * 10 + [_F, _I, _I, _P],
     "asb_differential_combine": [_P, _P, _I, _I, _I, _F, _F, _F, _I, _P],

@@ -42,19 +42,22 @@ class PageSpec:
     """What a mixer keeps in pages: the tensors each page holds, and what lets pages go early:
     `window` (only the last `window` positions are ever read) and `chunk` (a position reads only
     its own run of `chunk` positions, counted from the request's start), so older pages can be
-    given back before the request ends. Entries of the run order with equal specs share a group of
+    given back before the request ends; the pages of the first `keep_first` positions, which every
+    later position reads, are not. Entries of the run order with equal specs share a group of
     pools, an allocator and the requests' block tables."""
 
     tensors: tuple[PageTensor, ...]
     window: int | None = None
     chunk: int | None = None
+    keep_first: int = 0
 
     @property
     def values_per_token(self) -> int:
         return sum(t.heads * t.width for t in self.tensors)
 
     def first_needed(self, start: int) -> int:
-        """The lowest position that a step starting at position `start` can still read."""
+        """The lowest position, the kept first ones aside, that a step starting at position `start`
+        can still read."""
         lowest = 0
         if self.window is not None:
             lowest = max(lowest, start - self.window + 1)
@@ -63,10 +66,11 @@ class PageSpec:
         return lowest
 
 
-def KVCacheSpec(num_kv_heads: int, head_dim: int, window: int | None = None, chunk: int | None = None) -> PageSpec:
+def KVCacheSpec(num_kv_heads: int, head_dim: int, window: int | None = None, chunk: int | None = None,
+                keep_first: int = 0) -> PageSpec:  # fmt: skip
     """The usual pages: keys and values, `num_kv_heads * head_dim` of each per token, as tensors
     "k" and "v"."""
-    return PageSpec((PageTensor("k", num_kv_heads, head_dim), PageTensor("v", num_kv_heads, head_dim)), window, chunk)
+    return PageSpec((PageTensor("k", num_kv_heads, head_dim), PageTensor("v", num_kv_heads, head_dim)), window, chunk, keep_first)
 
 
 @dataclass(frozen=True)
@@ -325,6 +329,6 @@ def build_block(kind: str, mixer: Mixer, feed_forward: FeedForward, mixer_norm: 
 def _ensure_builtin() -> None:
     if "rms_norm" not in _REGISTRIES["norm"]:
         from atomserve_b200.parts import (  # noqa: F401
-            attention, block, differential_attention, embedding, experts, latent_attention, lightning, matrix_memory, mlp,
+            attention, block, differential_attention, embedding, experts, latent_attention, lightning, matrix_memory, mixed_heads, mlp,
             norms, parallel, rotary, sink_attention, state_space, stream_step, token_input,
         )

@@ -115,6 +115,10 @@ class SandwichNormBlock(PostNormBlock):
     the place where pre-norm blocks hand it on. Sublayers give their last product as float32 or as
     partial sums (`forward_for_stream`); a feed-forward's `output_bias` joins it before the norm."""
 
+    def feed_forward_output(self, h: torch.Tensor, ctx: StepContext):
+        ff = getattr(self.feed_forward, "forward_for_stream", None)
+        return ff(h, ctx) if ff is not None else self.feed_forward.forward(h, None, ctx)
+
     def forward_chain(self, x: torch.Tensor, normed: torch.Tensor | None, ctx: StepContext, cache: CacheView | None,
                       write_cache: bool, then: Norm | None) -> tuple[torch.Tensor, torch.Tensor | None]:  # fmt: skip
         h = normed if normed is not None else self.mixer_norm.forward(x)
@@ -123,9 +127,21 @@ class SandwichNormBlock(PostNormBlock):
         if not self.has_feed_forward:
             return self.mixer_norm.add_forward(x, y, then)
         x, h = self.mixer_norm.add_forward(x, y, self.feed_forward_norm)
-        ff = getattr(self.feed_forward, "forward_for_stream", None)
-        y = ff(h, ctx) if ff is not None else self.feed_forward.forward(h, None, ctx)
-        return self.feed_forward_norm.add_forward(x, y, then, getattr(self.feed_forward, "output_bias", None))
+        return self.feed_forward_norm.add_forward(x, self.feed_forward_output(h, ctx), then, getattr(self.feed_forward, "output_bias", None))
+
+
+class HyperConnectionBlock(SandwichNormBlock):
+    """The arrangement over several parallel residual streams: each sublayer reads a weighted sum of
+    them and its output goes back to all of them while they are mixed with one another. The norms are
+    `HyperConnection`s, which carry the streams' weights; the kernel that closes one sublayer opens the
+    next, so the flow is the one above, the streams [tokens, S, width] in the place of the one stream.
+    Routed experts hand over their rows and weights (`routed`), which that kernel sums up itself. A
+    model of such blocks ends in a norm that joins the streams (`StreamSumNorm`)."""
+
+    def feed_forward_output(self, h: torch.Tensor, ctx: StepContext):
+        if getattr(self.feed_forward, "sums_alone", None) is not None and self.feed_forward.sums_alone():
+            return self.feed_forward.routed(h)[0]
+        return super().feed_forward_output(h, ctx)
 
 
 class ParallelResidualBlock(PostNormBlock):
@@ -165,6 +181,7 @@ class ParallelResidualBlock(PostNormBlock):
         self.mixer_norm.block_norms = self.norms  # how the block before this one learns both gains
 
 
+register_part("block", "hyper_connections", HyperConnectionBlock)
 register_part("block", "parallel_residual", ParallelResidualBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)

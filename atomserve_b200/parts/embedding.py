@@ -69,13 +69,17 @@ class PairHashEmbedding(TokenEmbedding):
     a hashed table of token pairs beside the token table. `pairs` has buckets + 1 rows; the last
     one serves a sequence's first token, which has no predecessor. The token before a step's first
     one is kept per request as state (`last`: that id plus one, 0 after admission), so prompts may
-    be cut anywhere and decoded tokens know their predecessor without the host's help."""
+    be cut anywhere and decoded tokens know their predecessor without the host's help. With `norm_eps`
+the sum is then normed with a gain (`norm_tensor`), centred or not."""
 
     state_in_graphs = True  # one int per request, saved and put back around a capture's warm-up run
 
     def __init__(self, hidden_size: int, prefix: str, vocab_size: int, buckets: int, mul_prev: int, mul_cur: int,
-                 tensor: str | None = None, pair_tensor: str | None = None):  # fmt: skip
+                 tensor: str | None = None, pair_tensor: str | None = None, norm_eps: float | None = None,
+                 norm_tensor: str | None = None, norm_centred: bool = True):  # fmt: skip
         super().__init__(hidden_size, prefix, vocab_size, tensor)
+        self.norm_eps, self.norm_name, self.norm_centred = norm_eps, norm_tensor or prefix + "norm", norm_centred
+        self.gain: torch.Tensor | None = None
         if buckets < 1:
             raise ValueError(f"a pair table needs at least one bucket, got {buckets}")
         # (a x) mod b = ((a mod b) x) mod b: the multipliers go to the kernel reduced, whatever their size
@@ -84,11 +88,16 @@ class PairHashEmbedding(TokenEmbedding):
         self.pairs: torch.Tensor | None = None
 
     def tensor_specs(self) -> list[TensorSpec]:
-        return super().tensor_specs() + [TensorSpec(self.pair_name, (self.buckets + 1, self.hidden_size))]
+        specs = super().tensor_specs() + [TensorSpec(self.pair_name, (self.buckets + 1, self.hidden_size))]
+        if self.norm_eps is not None:
+            specs.append(TensorSpec(self.norm_name, (self.hidden_size,), kind="gain", init="gain"))
+        return specs
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         super().load(tensors)
         self.pairs = tensors[self.pair_name]
+        if self.norm_eps is not None:
+            self.gain = tensors[self.norm_name]
 
     def state_specs(self) -> list[StateSpec]:
         return [StateSpec("last", (1,), torch.int32)]
@@ -99,8 +108,11 @@ class PairHashEmbedding(TokenEmbedding):
     def forward_step(self, ctx: StepContext, cache: CacheView | None) -> torch.Tensor:
         if cache is None or "last" not in cache.state:
             raise RuntimeError("a pair embedding needs its per-request state")
-        return ops.pair_embedding(ctx.token_ids, ctx.positions, ctx.req_q_start, ctx.state_slots, cache.state["last"],
-                                  self.table, self.pairs, self.mul_prev, self.mul_cur, self.status)  # fmt: skip
+        x = ops.pair_embedding(ctx.token_ids, ctx.positions, ctx.req_q_start, ctx.state_slots, cache.state["last"],
+                               self.table, self.pairs, self.mul_prev, self.mul_cur, self.status)  # fmt: skip
+        if self.norm_eps is None:
+            return x
+        return ops.residual_out_norm(None, x, self.gain, self.norm_eps, torch.float32, centred=self.norm_centred)[0]
 
 
 class LMHead(Part):

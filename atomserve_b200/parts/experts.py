@@ -58,11 +58,15 @@ class GeluMLP(FeedForward):
 
 
 class RoutedExperts(FeedForward):
+    """Parameters beyond those named above: `score="chosen_softmax"`: the `top` largest logits win and
+    are weighted by their softmax among themselves; `router_bias`: the logits have a bias (`router.b`);
+    `form="relu2"`: an expert is down(max(up h, 0)^2), without a gate."""
+
     def __init__(self, hidden_size: int, prefix: str, experts: int, top: int, expert_ff: int, limit: float = 0.0,
                  groups: int = 1, group_top: int = 2, keep: int = 1, scale: float = 1.0, slope: float = 1.0,
                  shift: float = 0.0, score: str = "sigmoid", renormalise: bool = True, shared_ff: int | None = None,
                  shared_limit: float | None = None, shared_gated: bool = True, identity: int = 0,
-                 choice_offsets: bool = False):  # fmt: skip
+                 choice_offsets: bool = False, router_bias: bool = False, form: str = "clamped_glu"):  # fmt: skip
         # `identity`: that many further router outputs are experts without tensors whose output is their
         # input; `choice_offsets`: a learned vector (`correction`) joins the scores when the experts are
         # chosen and stays out of their weights
@@ -71,8 +75,17 @@ class RoutedExperts(FeedForward):
             raise ValueError("identity experts belong to no group of experts")
         if experts % groups or not 1 <= keep <= groups or not 1 <= top <= (experts + self.identity) // groups * keep:
             raise ValueError(f"{experts} experts in {groups} groups, {keep} kept, cannot give {top} choices")
-        if score not in ("sigmoid", "softmax"):
-            raise ValueError(f"score {score!r} is neither 'sigmoid' nor 'softmax'")
+        if score not in ("sigmoid", "softmax", "chosen_softmax"):
+            raise ValueError(f"score {score!r} is none of 'sigmoid', 'softmax' and 'chosen_softmax'")
+        if form not in ("clamped_glu", "relu2"):
+            raise ValueError(f"experts of form {form!r} are neither 'clamped_glu' nor 'relu2'")
+        if (score == "chosen_softmax") and (groups != 1 or choice_offsets or shared_gated and shared_ff is not None):
+            raise ValueError("a softmax over the chosen logits goes with one group, no selection offsets and no gated shared expert")
+        if router_bias and score != "chosen_softmax":
+            raise ValueError("a router bias goes with a softmax over the chosen logits")
+        if form == "relu2" and shared_ff is not None:
+            raise ValueError("experts without a gate have no shared expert")
+        self.router_bias, self.form = bool(router_bias), form
         self.hidden_size, self.prefix = hidden_size, prefix
         self.experts, self.top, self.expert_ff, self.limit = experts, top, expert_ff, float(limit)
         self.groups, self.group_top, self.keep, self.scale = groups, group_top, keep, float(scale)
@@ -85,7 +98,11 @@ class RoutedExperts(FeedForward):
         p, d, f = self.prefix, self.hidden_size, self.expert_ff
         specs = []
         for e in range(self.experts):
-            specs += [TensorSpec(f"{p}e{e}.gate", (f, d)), TensorSpec(f"{p}e{e}.up", (f, d)), TensorSpec(f"{p}e{e}.down", (d, f))]
+            if self.form == "clamped_glu":
+                specs.append(TensorSpec(f"{p}e{e}.gate", (f, d)))
+            specs += [TensorSpec(f"{p}e{e}.up", (f, d)), TensorSpec(f"{p}e{e}.down", (d, f))]
+        if self.router_bias:
+            specs.append(TensorSpec(p + "router.b", (self.experts + self.identity,), kind="gain", init="normal"))
         specs.append(TensorSpec(p + "router", (self.experts + self.identity, d)))
         if self.choice_offsets:
             specs.append(TensorSpec(p + "correction", (self.experts + self.identity,), kind="gain", init="normal"))
@@ -98,7 +115,8 @@ class RoutedExperts(FeedForward):
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         p, E = self.prefix, self.experts
-        self.gate = torch.stack([tensors[f"{p}e{e}.gate"] for e in range(E)]).contiguous()  # [E, F, d]
+        if self.form == "clamped_glu":
+            self.gate = torch.stack([tensors[f"{p}e{e}.gate"] for e in range(E)]).contiguous()  # [E, F, d]
         self.up = torch.stack([tensors[f"{p}e{e}.up"] for e in range(E)]).contiguous()
         self.down = torch.stack([tensors[f"{p}e{e}.down"] for e in range(E)]).contiguous()  # [E, d, F]
         rows = [tensors[p + "router"]]
@@ -109,19 +127,33 @@ class RoutedExperts(FeedForward):
             self.shared_down = tensors[p + "shared.down"]
         self.router = torch.cat(rows).contiguous()
         self.offsets = tensors[p + "correction"].contiguous() if self.choice_offsets else None
+        if self.router_bias:
+            self.offsets = tensors[p + "router.b"].contiguous()
 
-    def forward(self, h: torch.Tensor, residual: torch.Tensor | None, ctx: StepContext) -> torch.Tensor:
-        E, routed = self.experts, self.experts + self.identity
+    def routed(self, h: torch.Tensor) -> tuple[ops.ExpertSums, torch.Tensor, torch.Tensor | None]:
+        """(the chosen experts' outputs before their weighted sum, the choices, the shared expert's gate)."""
+        routed = self.experts + self.identity
         z = ops.linear(h, self.router, out_dtype=torch.float32)
         ids, weights, shared_gate = ops.route(
             z, experts=routed, top=self.top, groups=self.groups, group_top=self.group_top, keep=self.keep, scale=self.scale,
-            gate_col=routed if self.shared_gated else None, softmax=self.score == "softmax", renormalise=self.renormalise,
+            gate_col=routed if self.shared_gated else None, softmax="chosen" if self.score == "chosen_softmax" else self.score == "softmax", renormalise=self.renormalise,
             bias=self.offsets,
         )  # fmt: skip
         # (the identity experts' pairs are sorted behind the last expert's rows, where no product looks)
         offsets, row_token, pair_row = ops.group_by_expert(ids, routed)
-        hidden = ops.experts_glu(h, row_token, offsets, self.gate, self.up, self.limit, self.slope, self.shift)
-        y = ops.experts_down(hidden, offsets, self.down)
+        if self.form == "relu2":
+            hidden = ops.experts_relu2(h, row_token, offsets, self.up)
+        else:
+            hidden = ops.experts_glu(h, row_token, offsets, self.gate, self.up, self.limit, self.slope, self.shift)
+        return ops.ExpertSums(ops.experts_down(hidden, offsets, self.down), pair_row, weights), ids, shared_gate
+
+    def sums_alone(self) -> bool:
+        """Whether the layer's output is the routed experts' weighted sum and nothing else."""
+        return not self.identity and self.shared_ff is None
+
+    def forward(self, h: torch.Tensor, residual: torch.Tensor | None, ctx: StepContext) -> torch.Tensor:
+        sums, ids, shared_gate = self.routed(h)
+        y, pair_row, weights, E = sums.y, sums.pair_row, sums.weights, self.experts
         shared = None
         if self.shared_ff is not None:
             inner = ops.clamped_glu(ops.linear(h, self.shared_gate_up), self.shared_limit, self.slope, self.shift)

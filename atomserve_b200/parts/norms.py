@@ -143,6 +143,75 @@ class SandwichNorm(Norm):
         return ops.add_normed(x, y, self.out_gain, self.eps, gain_next, then.eps if then is not None else 0.0, self.dtype, bias)
 
 
+class HyperConnection(Norm):
+    """How one sublayer f hangs on S parallel residual streams (float32 [tokens, S, width]):
+    u = sum_s in[s] x_s is its input before the norm, and x_t <- sum_s mix[s, t] x_s + out[t] f(N(u))
+    what it leaves, N the centred norm (`centred=False`: the RMS norm) with a gain. `forward` is N(u) of
+    (rows of) the streams in the compute dtype; `add_forward(x, y, then, bias)` the new streams for the
+    sublayer's output y (+ bias) and, where `then` (the connection whose input comes next) is given,
+    that one's N(u) of them, from one kernel. `tensor` names the gain, `hc` the prefix of the three
+    tensors `in`, `out` [S] and `mix` [S, S] ([from, to]). A stream tensor [tokens, width], as an
+    embedding gives it, stands for S equal streams."""
+
+    def __init__(self, hidden_size: int, prefix: str, eps: float, streams: int, centred: bool = True, tensor: str | None = None,
+                 hc: str | None = None):  # fmt: skip
+        self.width, self.eps, self.streams, self.centred = hidden_size, float(eps), int(streams), bool(centred)
+        self.name, self.hc = tensor or prefix + "weight", hc or prefix + "hc."
+        self.gain = self.w_in = self.w_out = self.w_mix = None
+        self.dtype = torch.float32
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        S = self.streams
+        return [TensorSpec(self.name, (self.width,), kind="gain", init="gain"),
+                TensorSpec(self.hc + "in", (S,), kind="gain", init="gain"), TensorSpec(self.hc + "out", (S,), kind="gain", init="gain"),
+                TensorSpec(self.hc + "mix", (S, S), kind="gain", init="identity")]  # fmt: skip
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        self.gain = tensors[self.name]
+        self.w_in, self.w_out, self.w_mix = (tensors[self.hc + n].contiguous() for n in ("in", "out", "mix"))
+
+    def bind_dtype(self, dtype: torch.dtype) -> None:
+        self.dtype = dtype
+
+    def _streams(self, x: torch.Tensor) -> torch.Tensor:
+        return x if x.dim() == 3 else x.unsqueeze(1).expand(-1, self.streams, -1)
+
+    def forward(self, x: torch.Tensor, rows: torch.Tensor | None = None) -> torch.Tensor:
+        return ops.hyper_streams(self._streams(x), w_in=self.w_in, gain=self.gain, eps=self.eps, centred=self.centred,
+                                 dtype=self.dtype, rows=rows)[1]  # fmt: skip
+
+    def add_forward(self, x: torch.Tensor, y, then: Norm | None = None, bias: torch.Tensor | None = None):
+        if not isinstance(then, HyperConnection):
+            streams, _ = ops.hyper_streams(self._streams(x), y, w_out=self.w_out, w_mix=self.w_mix, bias=bias)
+            return streams, (then.forward(streams) if then is not None else None)
+        return ops.hyper_streams(self._streams(x), y, w_out=self.w_out, w_mix=self.w_mix, bias=bias, w_in=then.w_in, gain=then.gain,
+                                 eps=then.eps, centred=then.centred, dtype=self.dtype)  # fmt: skip
+
+
+class StreamSumNorm(Norm):
+    """A final norm over parallel residual streams: N(sum_s x_s) * gain of (rows of) them in the
+    compute dtype, N the centred norm or (`centred=False`) the RMS norm."""
+
+    def __init__(self, hidden_size: int, prefix: str, eps: float, streams: int, centred: bool = True, tensor: str | None = None):
+        self.width, self.eps, self.streams, self.centred = hidden_size, float(eps), int(streams), bool(centred)
+        self.name = tensor or prefix + "weight"
+        self.gain = self.ones = None
+        self.dtype = torch.float32
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        return [TensorSpec(self.name, (self.width,), kind="gain", init="gain")]
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        self.gain = tensors[self.name]
+        self.ones = torch.ones(self.streams, dtype=torch.float32, device=self.gain.device)
+
+    def bind_dtype(self, dtype: torch.dtype) -> None:
+        self.dtype = dtype
+
+    def forward(self, x: torch.Tensor, rows: torch.Tensor | None = None) -> torch.Tensor:
+        return ops.hyper_streams(x, w_in=self.ones, gain=self.gain, eps=self.eps, centred=self.centred, dtype=self.dtype, rows=rows)[1]
+
+
 class NoNorm(Norm):
     """The norm of a sublayer that a layer does not have."""
 
@@ -158,4 +227,6 @@ register_part("norm", "scaled_rms_norm", ScaledRMSNorm)
 register_part("norm", "stream_rms_norm", StreamRMSNorm)
 register_part("norm", "output_norm", OutputNorm)
 register_part("norm", "sandwich_norm", SandwichNorm)
+register_part("norm", "hyper_connection", HyperConnection)
+register_part("norm", "stream_sum_norm", StreamSumNorm)
 register_part("norm", "none", NoNorm)

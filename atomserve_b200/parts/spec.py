@@ -18,7 +18,7 @@ class TensorSpec:
           "gain"    a norm gain or other small vector; kept in float32 whatever it is stored as
           "int"     an integer table; kept as int32
     init: how the random-weights mode fills it: "normal" N(0, 0.02), "gain" 1 + N(0, 0.1),
-          "zeros", or "index" (integers below `high`).
+          "identity" the identity plus N(0, 0.1), "zeros", or "index" (integers below `high`).
     """
 
     name: str

@@ -1,7 +1,7 @@
 """Seeded random weights: for a model in memory, or written out as a model folder
 (config.json + model.safetensors) that the ordinary loader then reads.
 
-Matrices are N(0, 0.02), norm gains 1 + N(0, 0.1). Every tensor has its own generator seeded
+Matrices are N(0, 0.02), norm gains 1 + N(0, 0.1), small mixing matrices 1 + N(0, 0.1). Every tensor has its own generator seeded
 from (seed, tensor name), so a tensor's values do not depend on which other tensors exist or
 in which order they are made. (The reference has random weights only in its tests,
 tests/conftest.py:45-70.)
@@ -35,6 +35,8 @@ def random_tensor(spec: TensorSpec, seed: int, dtype: torch.dtype, device: torch
         t = torch.randn(spec.shape, generator=g, device=device, dtype=torch.float32) * 0.02
     elif spec.init == "gain":
         t = 1.0 + torch.randn(spec.shape, generator=g, device=device, dtype=torch.float32) * 0.1
+    elif spec.init == "identity":
+        t = torch.eye(*spec.shape, device=device) + torch.randn(spec.shape, generator=g, device=device, dtype=torch.float32) * 0.1
     elif spec.init == "zeros":
         t = torch.zeros(spec.shape, device=device, dtype=torch.float32)
     elif spec.init == "index":
