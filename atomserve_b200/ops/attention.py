@@ -135,13 +135,14 @@ def paged_attention(
 
     bfloat16 with head size 64 or 128 runs the tensor-core kernels (decode kernel for requests
     that bring at most 8 tokens, prefill kernel for longer portions; `host_q_lens`, the tokens
-    each request brings, tells which are needed); everything else, and `generic=True`, runs the
+    each request brings, tells which are needed; heads with a vector per key head have kernels of
+    their own); everything else, and `generic=True`, runs the
     general CUDA-core kernel.
     """
     require_cuda(q, k_cache, v_cache, block_tables, req_q_start, req_pos_start)
     KV, bs = k_cache.shape[1], k_cache.shape[2]
-    parts = 1
-    if q.dim() == 4:
+    parts, summed = 1, q.dim() == 4  # (with one kv head the sum has one term)
+    if summed:
         parts = q.shape[2]
         if parts != KV:
             raise KernelLibraryError(f"paged_attention: queries of {parts} parts against {KV} key heads")
@@ -162,9 +163,12 @@ def paged_attention(
             raise KernelLibraryError(f"paged_attention: sink must be contiguous float32 [{H}]")
     span = min(win, chunk) if win and chunk else (win or chunk)  # a chunk bounds the keys of a row as a window does
     keep = int(keep_first) if span else 0
-    if q.dtype == torch.bfloat16 and not generic and parts == 1 and not keep and lib().asb_attention_mma_supported(hd, H // KV):
+    if q.dtype == torch.bfloat16 and not generic and not summed and not keep and lib().asb_attention_mma_supported(hd, H // KV):
         return _paged_attention_mma(q, out, k_cache, v_cache, block_tables, req_q_start, req_pos_start,
                                     num_requests, max_context, win, scale, partitions, host_q_lens, sink, chunk, softcap, span)  # fmt: skip
+    if q.dtype == torch.bfloat16 and not generic and summed and not chunk and not softcap and sink is None and lib().asb_attention_parts_supported(hd, KV):
+        return _paged_attention_parts(q, out, k_cache, v_cache, block_tables, req_q_start, req_pos_start, num_requests, max_context,
+                                      win, keep, scale, partitions, host_q_lens)  # fmt: skip
     ps, np_ = partitions or plan_partitions(T, num_requests, KV, H // KV, max_context, span)
     part_m = part_l = part_acc = None
     if np_ > 1:
@@ -268,4 +272,71 @@ def _paged_attention_mma(q, out, k_cache, v_cache, block_tables, req_q_start, re
     if np_ > 1:
         check(lib().asb_attention_reduce(ptr(out), ptr(part_m), ptr(part_l), ptr(part_acc), T * H, np_, hd,
                                          dtype_code(q), stream()))  # fmt: skip
+    return out
+
+
+@functools.lru_cache(maxsize=4096)
+def plan_parts_partitions(rows: int, heads: int, kv_heads: int, max_context: int, window: int, keep: int, head_dim: int) -> tuple[int, int]:
+    """(key tiles of 64 per partition, partitions) for the decode kernel of heads with a vector per
+    key head, one block per (row, up to 16 heads, partition): the same weighing as
+    `plan_decode_partitions`, a tile's cost being the key and value heads that the block walks."""
+    per_block = lib().asb_attention_parts_heads(heads, kv_heads)
+    chunks = -(-heads // per_block)
+    resident = lib().asb_attention_parts_resident(head_dim, kv_heads) or 148
+    tiles = -(-max_context // 64)
+    if window:
+        tiles = min(tiles, -(-min(keep, max_context) // 64) + -(-window // 64) + 1)
+    items = (kv_heads + -(-kv_heads // chunks)) / 2  # a key head and a value head count as one tile of the plain kernel
+    best = None
+    for parts in range(1, min(tiles, 64) + 1):
+        size = -(-tiles // parts)
+        parts = -(-tiles // size)
+        cost = -(-rows * chunks * parts // resident) * (size * items + 3) + 0.5 * parts
+        if best is None or cost < best[0]:
+            best = (cost, size, parts)
+    return best[1], best[2]
+
+
+def _paged_attention_parts(q, out, k_cache, v_cache, block_tables, req_q_start, req_pos_start, num_requests, max_context, win, keep,
+                           scale, partitions, host_q_lens):  # fmt: skip
+    T, H, KV, hd = q.shape
+    bs = k_cache.shape[2]
+    lens = host_q_lens
+    has_short = lens is None or any(n <= SHORT_ROWS for n in lens)
+    has_long = lens is None or any(n > SHORT_ROWS for n in lens)
+    all_single = lens is not None and all(n == 1 for n in lens)
+    short_rows = T if lens is None else sum(n for n in lens if n <= SHORT_ROWS)
+
+    def launch(decode, long, pt, np_, m, l, acc, compact):
+        check(lib().asb_attention_parts(
+            ptr(out), ptr(q), ptr(k_cache), ptr(v_cache), ptr(block_tables), ptr(req_q_start), ptr(req_pos_start), ptr(m), ptr(l), ptr(acc),
+            T, num_requests, H, KV, hd, bs, block_tables.shape[1], win, keep, pt, np_, float(scale), int(decode), int(long),
+            int(all_single), compact, stream()))  # fmt: skip
+
+    if has_long and PREFILL_KERNEL == "tcgen05" and scale > 0 and lib().asb_attention_parts_tcgen05_supported(hd, H // KV, bs):
+        from atomserve_b200.ops.linear import gemm_status
+
+        check(lib().asb_attention_parts_tcgen05(
+            ptr(out), ptr(q), ptr(k_cache), ptr(v_cache), ptr(block_tables), ptr(req_q_start), ptr(req_pos_start), T, num_requests, H, KV, hd,
+            bs, k_cache.shape[0], block_tables.shape[1], win, keep, float(scale), ptr(gemm_status(q.device)), stream()))  # fmt: skip
+    elif has_long:
+        launch(False, True, 1, 1, None, None, None, 0)
+    if has_short:
+        # a step that also holds long portions starts blocks, and holds partial results, for the short rows only
+        compact = short_rows if has_long and lens is not None else 0
+        rows = compact or T
+        pt, np_ = partitions or plan_parts_partitions(short_rows, H, KV, max_context, win, keep, hd)
+        if partitions is None and (lens is None or rows * H * np_ * (hd + 2) * 4 > MIXED_SCRATCH_BYTES):
+            pt, np_ = 1 << 24, 1
+        m = l = acc = None
+        if np_ > 1:
+            m = torch.empty(rows * H * np_, device=q.device, dtype=torch.float32)
+            l = torch.empty_like(m)
+            acc = torch.empty(rows * H * np_ * hd, device=q.device, dtype=torch.float32)
+        launch(True, False, pt, np_, m, l, acc, compact)
+        if np_ > 1 and compact:
+            check(lib().asb_attention_reduce_short(ptr(out), ptr(m), ptr(l), ptr(acc), ptr(req_q_start), num_requests, SHORT_ROWS, compact,
+                                                   H, np_, hd, dtype_code(q), stream()))  # fmt: skip
+        elif np_ > 1:
+            check(lib().asb_attention_reduce(ptr(out), ptr(m), ptr(l), ptr(acc), T * H, np_, hd, dtype_code(q), stream()))
     return out

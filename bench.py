@@ -1064,6 +1064,124 @@ def time_nipurax(widths: list[int], layers: int, steps: int, warmup: int, pk: di
         print(json.dumps(line), flush=True)
 
 
+# ---- the Lidizen design beside Nipurax at equal width (`--only lidizen`) ---------------------------
+
+def lidizen_shape(width: int, layers: int) -> dict:
+    """Layer sizes that resemble a served model's: heads of 128 over four kv heads, half of every head
+    turned, four residual streams; layers with a window of 1,024 that keeps 16 positions alternate with
+    layers that see everything, and a dense feed-forward of three widths with 32 experts of the
+    width, 4 chosen."""
+    heads = width // 128
+    out = []
+    for i in range(layers):
+        m = dict(heads=heads, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, rot=dict(base=1000000.0, dims=64), v_mix=True)
+        if i % 2 == 0:
+            m["mask"] = dict(size=1024, keep_first=16)
+        mlp = dict(kind="moe", expert=dict(ff=width), router=dict(experts=32, top=4)) if i % 2 else dict(kind="dense", ff=3 * width)
+        out.append(dict(type="attention", mixer=m, mlp=mlp))
+    return dict(architecture="Lidizen", vocab=32000, width=width, streams=4, layers=out, norm=dict(eps=1e-6),
+                embedding=dict(bigram=dict(buckets=65521, mul_prev=1000003, mul_cur=31)))
+
+
+def time_lidizen(widths: list[int], layers: int, steps: int, warmup: int, pk: dict) -> None:
+    """Prefill and decode of a Lidizen model and of a Nipurax model of the same width and depth (random
+    weights), through the step function, and the design's own kernels one by one against their
+    rooflines beside the like kernels of the other models."""
+    import torch
+
+    from atomserve_b200 import ops
+
+    timed, model_times = design_timers(steps, warmup)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")  # noqa: E731
+    bw, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    bf = torch.bfloat16
+    for width in widths:
+        line = {"only": "lidizen", "width": width, "layers": layers, "peaks": pk["source"],
+                "lidizen": model_times(lidizen_shape(width, layers), 32000), "nipurax": model_times(nipurax_shape(width, layers), 32000)}
+        kern = {}
+        T, B, ctx, bs, S = PROMPT_TOKENS, 64, PROMPT_TOKENS, BLOCK_SIZE, 4
+        H, hd = width // 128, 128
+        pages_per = ctx // bs
+        tables = i32([[r * pages_per + j for j in range(pages_per)] for r in range(B)])
+        starts, at = i32(list(range(B + 1))), i32([ctx - 1] * B)
+        t1, whole, first = i32([list(range(pages_per))]), i32([0, T]), i32([0])
+        positions, slots = i32(list(range(T))), i32(list(range(T)))
+        # Attention. The design's arithmetic per visible (query head, key) pair: dim for the score, H for the mix,
+        # vdim for the values; the kernels multiply KV x dim + vdim (the mix lies in the queries). Beside it the plain
+        # causal attention at equal heads. Decode: the bytes of the keys and values a token sees.
+        for KV in (4, 8):
+            k_pages = torch.randn(B * pages_per, KV, bs, hd, device="cuda", dtype=bf)
+            v_pages = torch.randn_like(k_pages)
+            for name, mixed, window, keep in (("mixed_heads_attention", True, None, 0), ("mixed_heads_attention_windowed", True, 1024, 16),
+                                              ("paged_attention", False, None, 0), ("paged_attention_windowed", False, 1024, 0)):  # fmt: skip
+                part = (KV, hd) if mixed else (hd,)
+                more = dict(keep_first=keep) if mixed else {}
+                q = torch.randn(B, H, *part, device="cuda", dtype=bf)
+                keys = min(ctx, window + keep) if window else ctx
+                ms = timed(lambda: ops.paged_attention(q, k_pages, v_pages, tables, starts, at, num_requests=B, max_context=ctx, window=window,
+                                                       scale=0.03, host_q_lens=[1] * B, **more))  # fmt: skip
+                kern[f"{name}_kv{KV}_decode_b64"] = {"ms": round(ms, 4), "hbm_frac": round(2.0 * B * keys * KV * hd * 2 / (ms * 1e-3) / bw, 3)}
+                qp = torch.randn(T, H, *part, device="cuda", dtype=bf)
+                seen = sum(min(t + 1, keys) for t in range(T))
+                ms = timed(lambda: ops.paged_attention(qp, k_pages, v_pages, t1, whole, first, num_requests=1, max_context=T, window=window,
+                                                       scale=0.03, host_q_lens=[T], **more), 4)  # fmt: skip
+                design, done = (2 * hd + H, (KV + 1) * hd) if mixed else (2 * hd, 2 * hd)
+                kern[f"{name}_kv{KV}_prefill"] = {"ms": round(ms, 3), "tc_frac": round(2.0 * seen * H * design / (ms * 1e-3) / tf, 4),
+                                                  "tc_frac_multiplied": round(2.0 * seen * H * done / (ms * 1e-3) / tf, 4)}  # fmt: skip
+                del q, qp
+            # biases, norms, rotation, mix of the queries and of the values, page write; beside Qwen3's norm + rotation + page write
+            for rows, tag in ((T, "prefill"), (B, "decode_b64")):
+                proj = torch.randn(rows, (H + 2 * KV) * hd, device="cuda", dtype=bf)
+                bias, talk = torch.randn((H + 2 * KV) * hd, device="cuda"), torch.randn(H, H, device="cuda")
+                gq, gk, g1 = torch.ones(H * hd, device="cuda"), torch.ones(KV * hd, device="cuda"), torch.ones(hd, device="cuda")
+                inv = (1.0 / 1000000.0 ** (torch.arange(0, 64, 2, dtype=torch.float32) / 64)).cuda()
+                inv128 = (1.0 / 1000000.0 ** (torch.arange(0, hd, 2, dtype=torch.float32) / hd)).cuda()
+                v_first = torch.randn(rows, KV * hd, device="cuda", dtype=bf)
+                ms = timed(lambda: ops.mixed_heads_prepare(proj, H, KV, hd, hd, hd, positions[:rows], talk, bias=bias, q_gain=gq, k_gain=gk, eps=1e-6,
+                                                           inv_freq=inv, rotary_dim=64, v_first=v_first, lam=0.3, slots=slots[:rows],
+                                                           k_cache=k_pages, v_cache=v_pages))  # fmt: skip
+                moved = rows * (H + 5 * KV + H * KV) * hd * 2
+                kern[f"mixed_heads_prepare_kv{KV}_{tag}"] = {"ms": round(ms, 4), "hbm_frac": round(moved / (ms * 1e-3) / bw, 3)}
+                ms = timed(lambda: ops.qk_norm_rope_store(proj, H, KV, hd, positions[:rows], q_gain=g1, k_gain=g1, eps=1e-6, inv_freq=inv128,
+                                                          rotary_dim=hd, slots=slots[:rows], k_cache=k_pages, v_cache=v_pages))  # fmt: skip
+                kern[f"qk_norm_rope_store_kv{KV}_{tag}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * (2 * H + 4 * KV) * hd * 2 / (ms * 1e-3) / bw, 3)}
+            del k_pages, v_pages
+        # one sublayer closed and the next opened over the streams, beside Tigesun's norm after and before a sublayer
+        gain, vec, mix = torch.ones(width, device="cuda"), torch.ones(S, device="cuda"), torch.randn(S, S, device="cuda")
+        for name, rows in (("prefill", T), ("decode_b64", B)):
+            x, y = torch.randn(rows, S, width, device="cuda"), torch.randn(rows, width, device="cuda")
+            ms = timed(lambda: ops.hyper_streams(x, y, w_out=vec, w_mix=mix, bias=gain, w_in=vec, gain=gain, eps=1e-6, dtype=bf))
+            kern[f"hyper_streams_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * width * (8 * S + 6) / (ms * 1e-3) / bw, 3)}
+            ms = timed(lambda: ops.add_normed(y, y, gain, 1e-6, gain, 1e-6, bf, gain))
+            kern[f"add_normed_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * width * 14 / (ms * 1e-3) / bw, 3)}
+            # the experts: selection among biased logits; their weighted sum inside the streams' kernel, beside the
+            # weighted sum as a kernel of its own; and the grouped up products, without and with a gate
+            z, offsets = torch.randn(rows, 32, device="cuda"), torch.zeros(32, device="cuda")
+            ms = timed(lambda: ops.route(z, experts=32, top=4, softmax="chosen", bias=offsets))
+            kern[f"route_chosen_{name}"] = {"ms": round(ms, 4)}
+            ms = timed(lambda: ops.route(z, experts=32, top=4, scale=2.5, softmax=True, renormalise=False, bias=offsets))
+            kern[f"route_offsets_{name}"] = {"ms": round(ms, 4)}
+            ids, weights, _ = ops.route(z, experts=32, top=4, softmax="chosen", bias=offsets)
+            expert_offsets, row_token, pair_row = ops.group_by_expert(ids, 32)
+            out4 = torch.randn(rows * 4, width, device="cuda")
+            sums = ops.ExpertSums(out4, pair_row, weights)
+            ms = timed(lambda: ops.hyper_streams(x, sums, w_out=vec, w_mix=mix, w_in=vec, gain=gain, eps=1e-6, dtype=bf))
+            kern[f"hyper_streams_experts_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * width * (8 * S + 16 + 2) / (ms * 1e-3) / bw, 3)}
+            ms = timed(lambda: ops.combine(out4, pair_row, weights))
+            kern[f"combine_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * width * (4 * 4 + 4) / (ms * 1e-3) / bw, 3)}
+            ff = width // 2
+            h = torch.randn(rows, width, device="cuda", dtype=bf)
+            up, gate = torch.randn(32, 2 * ff, width, device="cuda", dtype=bf), torch.randn(32, ff, width, device="cuda", dtype=bf)
+            for which, fn in (("experts_relu2", lambda: ops.experts_relu2(h, row_token, expert_offsets, up)),
+                              ("experts_glu", lambda: ops.experts_glu(h, row_token, expert_offsets, gate, gate, 7.0, 1.702, 1.0))):  # fmt: skip
+                ms = timed(fn, 4)
+                kern[f"{which}_{name}"] = {"ms": round(ms, 4), "tc_frac": round(2.0 * rows * 4 * width * 2 * ff / (ms * 1e-3) / tf, 4),
+                                           "hbm_frac": round(32 * 2 * ff * width * 2 / (ms * 1e-3) / bw, 3)}  # fmt: skip
+            del up, gate
+        line["kernels"] = kern
+        print(json.dumps(line), flush=True)
+
+
 def tigesun_inner(width: int, ff: int, w_gu, b_gu):
     """A gated feed-forward part holding the given stacked gate and up rows ([2 ff, width], gate first)."""
     import torch
@@ -1131,7 +1249,7 @@ def main() -> int:
                         help="fewer layers than the model has (same layer sizes), where time or memory needs it")  # fmt: skip
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    parser.add_argument("--only", choices=["decode", "prefill", "gemm", "serve", "attention", "sampling", "designs", "zogepel", "tigesun", "nipurax"], help="time just this (for profiling small cases and the other shapes)")
+    parser.add_argument("--only", choices=["decode", "prefill", "gemm", "serve", "attention", "sampling", "designs", "zogepel", "tigesun", "nipurax", "lidizen"], help="time just this (for profiling small cases and the other shapes)")
     parser.add_argument("--shape", default="8b", choices=sorted(SHAPES), help="with --only decode/prefill/serve: layer sizes of Qwen3-8B, -14B or -32B")
     parser.add_argument("--context", type=int, default=PROMPT_TOKENS, help="with --only decode: tokens each request holds when decoding starts")
     parser.add_argument("--requests", type=int, default=32, help="with --only serve: requests submitted at once")
@@ -1139,7 +1257,7 @@ def main() -> int:
     parser.add_argument("--budget", type=int, default=512, help="with --only serve: the scheduler's token budget per step")
     parser.add_argument("--gemm-shape", default="all", help="with --only gemm: qkv, o, gate_up, down, lm_head or all")
     parser.add_argument("--gemm-tokens", default="1,8,64,2048", help="with --only gemm: token counts, comma-separated")
-    parser.add_argument("--widths", default="2048,4096", help="with --only designs, zogepel, tigesun or nipurax: model widths, comma-separated")
+    parser.add_argument("--widths", default="2048,4096", help="with --only designs, zogepel, tigesun, nipurax or lidizen: model widths, comma-separated")
     parser.add_argument("--timeline", action="store_true", help="with --only gemm: where a decode-size call's time goes")
     args = parser.parse_args()
     args.layers_given = any(a == "--layers" or a.startswith("--layers=") for a in sys.argv[1:])
@@ -1173,6 +1291,9 @@ def main() -> int:
         return 0
     if args.only == "nipurax":
         time_nipurax([int(w) for w in args.widths.split(",")], args.layers if args.layers_given else 4, max(args.steps // 4, 8), warmup, pk)
+        return 0
+    if args.only == "lidizen":
+        time_lidizen([int(w) for w in args.widths.split(",")], args.layers if args.layers_given else 4, max(args.steps // 4, 8), warmup, pk)
         return 0
     if args.only == "gemm" and args.timeline:
         gemm_timelines(args.gemm_shape, [int(t) for t in args.gemm_tokens.split(",")])

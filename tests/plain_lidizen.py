@@ -193,3 +193,75 @@ def forward(tokens: list[int], weights: dict, cfg: dict, streams: list | None = 
             streams.append(X.sum(1))
     x = stored(centred_norm(X.sum(1), weights["final.norm"], eps))
     return x @ weights["embed"].to(F64).T
+
+
+def tensor_shapes(cfg: dict) -> dict[str, tuple[int, ...]]:
+    """Names and shapes of a checkpoint (the factor of a layer that has nothing to mix its values with aside)."""
+    d, S = cfg["width"], cfg["streams"]
+    shapes = {"embed": (cfg["vocab"], d), "bigram": (cfg["embedding"]["bigram"]["buckets"] + 1, d), "embed.norm": (d,)}
+    mixed_before = False
+    for i, spec in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", spec["mixer"], spec.get("mlp")
+        H, G = m["heads"], m["kv_heads"]
+        rows = dict(q=H * m["dim"], k=G * m["dim"], v=G * m["vdim"])
+        for n, r in rows.items():
+            shapes[f"{p}mix.{n}"], shapes[f"{p}mix.{n}.b"] = (r, d), (r,)
+        shapes[p + "mix.q.norm"], shapes[p + "mix.k.norm"] = (rows["q"],), (rows["k"],)
+        shapes[p + "mix.talk"], shapes[p + "mix.o"] = (H, H), (d, H * m["vdim"])
+        if m.get("v_mix"):
+            if mixed_before:
+                shapes[p + "mix.vmix"] = ()
+            mixed_before = True
+        for q in (1, 2) if mlp is not None else (1,):
+            shapes[f"{p}norm{q}"] = (d,)
+            shapes[f"{p}hc{q}.in"], shapes[f"{p}hc{q}.out"], shapes[f"{p}hc{q}.mix"] = (S,), (S,), (S, S)
+        if mlp is None:
+            continue
+        if mlp["kind"] == "dense":
+            f = mlp["ff"]
+            shapes.update({p + "mlp.gate": (f, d), p + "mlp.gate.b": (f,), p + "mlp.up": (f, d), p + "mlp.up.b": (f,),
+                           p + "mlp.down": (d, f), p + "mlp.down.b": (d,)})  # fmt: skip
+        else:
+            E, f = mlp["router"]["experts"], mlp["expert"]["ff"]
+            for e in range(E):
+                shapes[f"{p}mlp.e{e}.up"], shapes[f"{p}mlp.e{e}.down"] = (f, d), (d, f)
+            shapes[p + "mlp.router"], shapes[p + "mlp.router.b"] = (E, d), (E,)
+    shapes["final.norm"] = (d,)
+    return shapes
+
+
+def random_checkpoint(cfg: dict, seed: int) -> dict[str, torch.Tensor]:
+    """Random float32 weights whose matrices are exact in bfloat16: matrices N(0, 1 / fan_in) (the two
+    embedding tables N(0, 1), routers N(0, 4 / fan_in) so that choices are seldom close), gains
+    1 + N(0, 0.1), biases N(0, 0.3), the mix of heads 1 + N(0, 0.25), the streams' weights away from one
+    another, the values' factor in 0.2 .. 0.7."""
+    g = torch.Generator().manual_seed(seed)
+    w = {}
+    for name, shape in tensor_shapes(cfg).items():
+        last = name.rsplit(".", 1)[-1]
+        noise = torch.randn(shape, generator=g)
+        if last == "vmix":
+            w[name] = 0.2 + 0.5 * torch.rand(shape, generator=g)
+        elif last == "talk":
+            w[name] = torch.eye(shape[0]) + 0.5 * shape[0] ** -0.5 * noise
+        elif ".hc" in name:
+            S = shape[0]
+            w[name] = {"in": 1.0 / S + 0.3 * noise, "out": 1.0 + 0.3 * noise, "mix": 0.8 * torch.eye(S) + 0.25 * noise if last == "mix" else None}[last]
+        elif last == "b":
+            w[name] = 0.3 * noise
+        elif len(shape) == 1:
+            w[name] = 1.0 + 0.1 * noise
+        else:
+            std = 1.0 if name in ("embed", "bigram") else (2.0 if last == "router" else 1.0) * shape[1] ** -0.5
+            w[name] = (noise * std).bfloat16().float()
+    return w
+
+
+def greedy_generate(tokens: list[int], weights: dict, cfg: dict, n: int) -> list[int]:
+    """The n tokens that follow when the largest logit is taken each time (the whole sequence is
+    run again for every token: slow and stateless)."""
+    tokens = list(tokens)
+    first = len(tokens)
+    for _ in range(n):
+        tokens.append(int(forward(tokens, weights, cfg)[-1].argmax()))
+    return tokens[first:]
