@@ -10,9 +10,10 @@
 // Q K^T is several times P V and the block is bound by the first product's operands and issue. Tiles of
 // 128 keys (rather than 64) halve the MMAs a score costs their issuing thread.
 //
-//   warp 0     TMA: the queries of all parts once (where they fit), then the keys in stages of
-//              [128 keys][64 entries of one part]; where the queries do not fit, each stage brings
-//              the matching [128 rows][64 entries] of them too.
+//   warps 0, 8 TMA: the queries of all parts once (where they fit), then the keys in stages of
+//              [128 keys][128 entries of one part], the two warps taking turns (a stage's wait,
+//              announcement and requests take a warp longer than the MMAs that read it); where the
+//              queries do not fit, each stage brings the part's [128 rows][128 entries] of them too.
 //   warp 7     TMA: the values, in stages of [64 keys][128 entries].
 //   warp 1     MMA: S[b] = sum over parts of Q_c K_c^T into score buffer b = tile & 1.
 //   warp 6     MMA: O += P V once the softmax has written P over the scores, where it is the A operand.
@@ -27,14 +28,15 @@ namespace {
 
 using namespace asb::t5;
 
-constexpr int kThreads = 256;
+constexpr int kThreads = 288;
 constexpr int HD = 128;
 constexpr int kRows = 128;
 constexpr int kKeys = 128;                       // keys per tile
 constexpr int kBlockBytes = 128 * 64 * 2;        // [128 rows][64 entries], swizzled: 16 KB
 constexpr int kVBlockBytes = 64 * 64 * 2;        // [64 keys][64 entries]: 8 KB
 constexpr int kVBytes = 2 * kVBlockBytes;        // a stage of values: 64 keys, both halves of the head
-constexpr int kVStages = 2, kMaxKStages = 8;
+constexpr int kVStages = 2, kMaxKStages = 4;
+constexpr int kKBytes = 2 * kBlockBytes;         // a stage of keys (or of queries): 128 rows, both halves of the head
 constexpr int kBarrierBytes = 256;
 constexpr int kMaxSmem = 227 * 1024;
 constexpr uint32_t kTmemCols = 512;
@@ -74,7 +76,7 @@ parts_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              const __grid_constant__ CUtensorMap map_v, const PartsParams p) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];  // the swizzled tiles need this alignment
   const uint32_t base = smem_u32(smem_raw);
-  constexpr int kStageBytes = kStreamQ ? 2 * kBlockBytes : kBlockBytes;
+  constexpr int kStageBytes = kStreamQ ? 2 * kKBytes : kKBytes;
   const int KS = p.k_stages;
   const uint32_t q_smem = base;  // [KV][2 halves] blocks, where they stay
   const uint32_t k_base = base + (kStreamQ ? 0u : (uint32_t)p.KV * 2u * kBlockBytes);
@@ -150,74 +152,81 @@ parts_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
   asb::pdl_wait();
   asb::pdl_launch_dependents();
 
-  if (warp == 0 || warp == 7) {
-    const bool keys = warp == 0;
-    const uint32_t q_bytes = (uint32_t)(p.QT * p.G * 128);  // a box of queries: QT x G rows, at most 128
-    if (keys && lane == 0 && !kStreamQ) {
+  const int last_page = (hi - 1) / p.bs;
+  const uint32_t q_bytes = (uint32_t)(p.QT * p.G * 128);  // a box of queries: QT x G rows, at most 128
+  // Pages beyond the request's end, or given back behind the window, are masked out anyway: a page the
+  // request holds is read instead, so that shared memory never holds non-finite values.
+  auto page_row = [&](int key) {  // row of kv head 0 in the pools
+    int blk = table[min(key / p.bs, last_page)];
+    if (blk < 0) blk = table[last_page];
+    return blk * p.KV * p.bs + key % p.bs;
+  };
+  if (warp == 0 || warp == 8) {
+    if (warp == 0 && lane == 0 && !kStreamQ) {
       mbar_expect_tx(q_full, 2u * p.KV * q_bytes);
       for (int c = 0; c < 2 * p.KV; ++c) tma_load_3d(q_smem + (uint32_t)c * kBlockBytes, &map_q, q_full, c * 64, head0, row0);
     }
-    const int box_rows = min(p.bs, keys ? kKeys : 64);             // rows one box brings
-    const int boxes = (keys ? kKeys : 64) / box_rows;              // at most 16 of keys, 8 of values
-    const int last_page = (hi - 1) / p.bs, fallback = table[last_page];
-    Ring ring;
-    bool ok = true;
-    for (int j = 0; j < num_tiles && ok; ++j) {
-      for (int sub = 0; sub < (keys ? 1 : 2) && ok; ++sub) {
-        // pages beyond the request's end, or given back behind the window, are masked out anyway: read
-        // a page the request holds, so that shared memory never holds non-finite values
-        int row_y = 0;
-        if (lane < boxes) {
-          const int key = first_key(j) + sub * 64 + lane * box_rows;
-          int blk = table[min(key / p.bs, last_page)];
-          if (blk < 0) blk = fallback;
-          row_y = (blk * p.KV + (keys ? 0 : kvh)) * p.bs + key % p.bs;
-        }
-        for (int item = 0; item < (keys ? 2 * p.KV : 1); ++item) {  // keys: both halves of every part
-          const int s = ring.stage;
-          int ok_i = 1;
-          if (lane == 0) {
-            ok_i = mbar_wait(keys ? k_empty(s) : v_empty(s), (ring.round & 1u) ^ 1u, p.status, keys ? 11 : 21) ? 1 : 0;
-            if (ok_i) mbar_expect_tx(keys ? k_full(s) : v_full(s), keys ? kBlockBytes + (kStreamQ ? q_bytes : 0u) : (uint32_t)kVBytes);
-          }
-          ok = __shfl_sync(0xffffffffu, ok_i, 0) != 0;
-          if (!ok) break;
-          if (keys) {
-            if (lane < boxes)
-              tma_load_2d(k_smem(s) + (uint32_t)(lane * box_rows) * 128u, &map_k, k_full(s), (item & 1) * 64, row_y + (item >> 1) * p.bs);
-            if (kStreamQ && lane == 31) tma_load_3d(k_smem(s) + kBlockBytes, &map_q, k_full(s), item * 64, head0, row0);
-          } else {
-            const int i = lane >> 1, which = lane & 1;
-            const int y = __shfl_sync(0xffffffffu, row_y, i);
-            if (i < boxes) tma_load_2d(v_smem(s) + (uint32_t)(i * box_rows) * 128u + (uint32_t)which * kVBlockBytes, &map_v, v_full(s), which * 64, y);
-          }
-          ring.next(keys ? KS : kVStages);
-        }
+    const int box_rows = min(p.bs, kKeys), boxes = kKeys / box_rows;  // rows one box brings; at most 16 boxes of each half
+    const int i = lane >> 1, which = lane & 1;                        // a lane's box and half
+    const int total = num_tiles * p.KV;
+    int row_y = 0, tile_of_row = -1;
+    for (int n = warp >> 3; n < total; n += 2) {
+      const int j = n / p.KV, c = n - j * p.KV, s = n % KS;
+      if (j != tile_of_row && i < boxes) row_y = page_row(first_key(j) + i * box_rows);
+      tile_of_row = j;
+      int ok_i = 1;
+      if (lane == 0) {
+        ok_i = mbar_wait(k_empty(s), ((uint32_t)(n / KS) & 1u) ^ 1u, p.status, 11) ? 1 : 0;
+        if (ok_i) mbar_expect_tx(k_full(s), (uint32_t)kKBytes + (kStreamQ ? 2u * q_bytes : 0u));
       }
+      if (!__shfl_sync(0xffffffffu, ok_i, 0)) break;
+      if (i < boxes)
+        tma_load_2d(k_smem(s) + (uint32_t)which * kBlockBytes + (uint32_t)(i * box_rows) * 128u, &map_k, k_full(s), which * 64, row_y + c * p.bs);
+      if (kStreamQ && lane < 2) tma_load_3d(k_smem(s) + kKBytes + (uint32_t)lane * kBlockBytes, &map_q, k_full(s), c * HD + lane * 64, head0, row0);
+    }
+  } else if (warp == 7) {
+    const int box_rows = min(p.bs, 64), boxes = 64 / box_rows;  // at most 8 boxes of each half
+    const int i = lane >> 1, which = lane & 1;
+    for (int n = 0; n < 2 * num_tiles; ++n) {
+      const int s = n % kVStages;
+      const int row_y = i < boxes ? page_row(first_key(n >> 1) + (n & 1) * 64 + i * box_rows) + kvh * p.bs : 0;
+      int ok_i = 1;
+      if (lane == 0) {
+        ok_i = mbar_wait(v_empty(s), ((uint32_t)(n / kVStages) & 1u) ^ 1u, p.status, 21) ? 1 : 0;
+        if (ok_i) mbar_expect_tx(v_full(s), (uint32_t)kVBytes);
+      }
+      if (!__shfl_sync(0xffffffffu, ok_i, 0)) break;
+      if (i < boxes) tma_load_2d(v_smem(s) + (uint32_t)which * kVBlockBytes + (uint32_t)(i * box_rows) * 128u, &map_v, v_full(s), which * 64, row_y);
     }
   } else if (warp == 1) {
     // S = Q K^T, a tile ahead of the softmax
     if (lane == 0) {
       constexpr uint32_t idesc_qk = instr_desc_bf16(kRows, kKeys, false);
       bool ok = kStreamQ || mbar_wait(q_full, 0, p.status, 12);
+      const int total = num_tiles * p.KV;
+      uint32_t there = 0;  // the answer to an early question about this stage (asking takes a few hundred cycles)
       Ring ring;
-      for (int j = 0; j < num_tiles && ok; ++j) {
+      for (int n = 0, j = 0, c = 0; n < total && ok; ++n) {
         // score buffer j & 1 held tile j - 2's scores and then its P: has that tile's P V read it?
-        if (j >= 2) ok = mbar_wait(pv_done(j & 1), ((uint32_t)(j - 2) >> 1) & 1u, p.status, 18);
-        for (int item = 0; item < 2 * p.KV && ok; ++item) {
-          const int s = ring.stage;
-          ok = mbar_wait(k_full(s), ring.round & 1u, p.status, 13);
-          if (!ok) break;
-          fence_after_sync();
-          const uint32_t q_block = kStreamQ ? k_smem(s) + kBlockBytes : q_smem + (uint32_t)item * kBlockBytes;
+        if (c == 0 && j >= 2) ok = mbar_wait(pv_done(j & 1), ((uint32_t)(j - 2) >> 1) & 1u, p.status, 18);
+        const int s = ring.stage;
+        if (ok && !there) ok = mbar_wait(k_full(s), ring.round & 1u, p.status, 13);
+        if (!ok) break;
+        fence_after_sync();
+        ring.next(KS);
+        there = n + 1 < total ? mbar_try(k_full(ring.stage), ring.round & 1u) : 0u;
+        const uint32_t q_block = kStreamQ ? k_smem(s) + kKBytes : q_smem + (uint32_t)c * kKBytes;
 #pragma unroll
-          for (int ks = 0; ks < 4; ++ks)  // 16 entries per MMA: 32 bytes along the swizzled row
-            umma_bf16(tmem_s(j), desc_k_major(q_block + (uint32_t)ks * 32u, 1024), desc_k_major(k_smem(s) + (uint32_t)ks * 32u, 1024),
-                      idesc_qk, (uint32_t)((item | ks) != 0));
-          umma_commit(k_empty(s));
-          ring.next(KS);
+        for (int ks = 0; ks < HD / 16; ++ks) {  // 16 entries per MMA: 32 bytes along the swizzled row
+          const uint32_t at = (uint32_t)(ks / 4) * kBlockBytes + (uint32_t)(ks % 4) * 32u;
+          umma_bf16(tmem_s(j), desc_k_major(q_block + at, 1024), desc_k_major(k_smem(s) + at, 1024), idesc_qk, (uint32_t)((c | ks) != 0));
         }
-        if (ok) umma_commit(s_full(j & 1));
+        umma_commit(k_empty(s));
+        if (++c == p.KV) {
+          umma_commit(s_full(j & 1));
+          c = 0;
+          ++j;
+        }
       }
     }
   } else if (warp == 6) {
@@ -369,9 +378,9 @@ parts_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
 
 // stages of keys that fit beside the queries of all parts; 0: too few, the queries travel with the keys
 int resident_stages(int KV) {
-  const int left = kMaxSmem - KV * 2 * kBlockBytes - kVStages * kVBytes - kBarrierBytes;
-  const int stages = left > 0 ? left / kBlockBytes : 0;
-  return stages >= 3 ? (stages < kMaxKStages ? stages : kMaxKStages) : 0;
+  const int left = kMaxSmem - KV * kKBytes - kVStages * kVBytes - kBarrierBytes;
+  const int stages = left > 0 ? left / kKBytes : 0;
+  return stages >= 2 ? (stages < kMaxKStages ? stages : kMaxKStages) : 0;
 }
 
 }  // namespace
@@ -405,8 +414,8 @@ extern "C" int asb_attention_parts_tcgen05(void* out, const void* q, const void*
   p.window = window; p.keep = window > 0 ? keep : 0;
   p.scale_log2 = scale * 1.4426950408889634f;
   const int stages = resident_stages(KV);
-  p.k_stages = stages ? stages : 4;
-  const int smem = (stages ? KV * 2 * kBlockBytes + stages * kBlockBytes : p.k_stages * 2 * kBlockBytes) + kVStages * kVBytes + kBarrierBytes;
+  p.k_stages = stages ? stages : 3;
+  const int smem = (stages ? (KV + stages) * kKBytes : p.k_stages * 2 * kKBytes) + kVStages * kVBytes + kBarrierBytes;
 
   alignas(64) CUtensorMap mq, mk, mv;
   {
