@@ -4,8 +4,8 @@
 // those of its own kv head h / G. Head sizes 64 and 128, any number of heads and kv heads, causal, with
 // an optional sliding window that may keep the sequence's first positions visible. Two kernels:
 //
-//   decode   one block per (new token, up to 16 query heads, key partition): the heads are the rows
-//            of a 16-row tile, so a key is read once for all of them. Per tile of 64 keys the block
+//   decode   one block per (new token, up to 32 query heads, key partition): the heads are the rows
+//            of one or two 16-row tiles, so a key is read once for all of them. Per tile of 64 keys the block
 //            walks the KV key heads, the scores growing in registers, and then the value heads that
 //            its rows belong to, each with the other rows' weights at zero. Four warps share a tile,
 //            sixteen keys apiece, and merge at the end. Serves requests of at most kShortRows tokens.
@@ -28,7 +28,7 @@ using namespace asb::mma;
 
 constexpr int kKeyTile = 64;
 constexpr int kShortRows = 8;  // requests with at most this many new tokens go row by row
-constexpr int kDecodeThreads = 128, kDecodeStages = 4;
+constexpr int kDecodeThreads = 128;
 constexpr int kPrefillThreads = 256, kPrefillRows = 128;
 
 struct PartsParams {
@@ -44,7 +44,7 @@ struct PartsParams {
   float* part_acc;               // [rows, H, NP, HD]
   int T, R, H, KV, bs, table_width;
   int G;                         // query heads per kv head
-  int GC, HC;                    // decode: heads per block (<= 16) and blocks; prefill: the same within a kv head
+  int GC, HC;                    // decode: heads per block (<= 32) and blocks; prefill: the same within a kv head
   int QT;                        // prefill: tokens per 128-row tile
   int window, keep;              // 0: none
   int PT, NP;                    // key tiles per partition, partitions (decode)
@@ -64,41 +64,54 @@ struct TileList {
   __device__ __forceinline__ int first_key(int t) const { return (t < kept ? t : t - kept + begin) * kKeyTile; }
 };
 
-// Keys (or values) kt0 .. kt0 + 63 of one kv head into a tile; positions no row sees are zero. A
-// thread copies one 16-byte column of a run of consecutive positions, looking a page up once where
-// the run lies inside one.
+// How a thread copies a tile of 64 keys (or values) of one kv head: one 16-byte column of a run of
+// consecutive positions. Where the run lies inside one page, the page is looked up once per tile, and
+// for the next tile while this one's heads are copied.
 template <int HD, int NT>
-__device__ __forceinline__ void load_tile(uint32_t tile, const __nv_bfloat16* cache, const PartsParams& p, const int* table,
-                                          int head, int kt0, int lo, int hi, int keep) {
-  constexpr int kChunks = HD / 8, kRun = kKeyTile / (NT / kChunks);
-  const int chunk = threadIdx.x % kChunks, run0 = (threadIdx.x / kChunks) * kRun, j0 = kt0 + run0;
-  const bool one_page = p.bs >= kRun && (p.bs & (p.bs - 1)) == 0;
-  auto seen = [&](int j) { return j < hi && (j >= lo || j < keep); };
-  size_t page_at = 0;
-  if (one_page && j0 < hi && (j0 + kRun > lo || j0 < keep))
-    page_at = (((size_t)table[j0 / p.bs] * p.KV + head) * p.bs + (j0 & (p.bs - 1))) * HD + chunk * 8;
-#pragma unroll
-  for (int i = 0; i < kRun; ++i) {
-    const int j = j0 + i;
-    const bool valid = seen(j);
-    size_t at = 0;
-    if (valid) at = one_page ? page_at + (size_t)i * HD : (((size_t)table[j / p.bs] * p.KV + head) * p.bs + j % p.bs) * HD + chunk * 8;
-    cp_async16(tile + tile_offset<HD>(run0 + i, chunk), cache + at, valid);
+struct TileCopy {
+  static constexpr int kChunks = HD / 8, kRun = kKeyTile / (NT / kChunks);
+  int chunk, run0, ahead = 0, block = 0;
+  bool one_page;
+
+  __device__ __forceinline__ TileCopy(const PartsParams& p)
+      : chunk(threadIdx.x % kChunks), run0(threadIdx.x / kChunks * kRun), one_page(p.bs >= kRun && (p.bs & (p.bs - 1)) == 0) {}
+
+  // ask for the page of the thread's run in the tile at kt0 (the answer is taken up by `enter`)
+  __device__ __forceinline__ void look(const PartsParams& p, const int* table, int kt0, int lo, int hi, int keep) {
+    const int j0 = kt0 + run0;
+    if (one_page && j0 < hi && (j0 + kRun > lo || j0 < keep)) ahead = table[j0 / p.bs];
   }
-}
+  __device__ __forceinline__ void enter() { block = ahead; }
+
+  // positions that no row sees are zero
+  __device__ __forceinline__ void load(uint32_t tile, const __nv_bfloat16* cache, const PartsParams& p, const int* table, int head,
+                                       int kt0, int lo, int hi, int keep) const {
+    const int j0 = kt0 + run0;
+    const size_t page_at = (((size_t)block * p.KV + head) * p.bs + (j0 & (p.bs - 1))) * HD + chunk * 8;
+#pragma unroll
+    for (int i = 0; i < kRun; ++i) {
+      const int j = j0 + i;
+      const bool valid = j < hi && (j >= lo || j < keep);
+      size_t at = 0;
+      if (valid) at = one_page ? page_at + (size_t)i * HD : (((size_t)table[j / p.bs] * p.KV + head) * p.bs + j % p.bs) * HD + chunk * 8;
+      cp_async16(tile + tile_offset<HD>(run0 + i, chunk), cache + at, valid);
+    }
+  }
+};
 
 // ---- decode ------------------------------------------------------------------------------------
 
-template <int HD>
+// MT: tiles of 16 query heads; NS: stages of the ring
+template <int HD, int MT, int NS>
 __global__ void __launch_bounds__(kDecodeThreads)
 parts_decode_kernel(const PartsParams p) {
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   extern __shared__ __align__(128) unsigned char smem_raw[];
-  constexpr int kTileBytes = kKeyTile * HD * 2, kQPart = 16 * HD * 2;
+  constexpr int kTileBytes = kKeyTile * HD * 2, kRows = 16 * MT, kQPart = kRows * HD * 2;
   const uint32_t smem = smem_u32(smem_raw);
-  auto stage = [&](int n) { return smem + (uint32_t)(n % kDecodeStages) * kTileBytes; };
-  const uint32_t q_tile = smem + kDecodeStages * kTileBytes;  // [KV][16 rows]
+  auto stage = [&](int n) { return smem + (uint32_t)(n % NS) * kTileBytes; };
+  const uint32_t q_tile = smem + NS * kTileBytes;  // [KV][kRows]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int row = blockIdx.x, r;
@@ -121,112 +134,144 @@ parts_decode_kernel(const PartsParams p) {
   const int t_begin = blockIdx.z * p.PT, t_end = min(tiles.count, t_begin + p.PT);
   const int total = max(0, t_end - t_begin) * items;
 
-  int load_tile_no = t_begin, load_item = 0, loaded = 0;
+  TileCopy<HD, kDecodeThreads> copy(p);
+  int load_kt0 = tiles.first_key(t_begin), next_kt0 = 0, load_tile_no = t_begin, load_item = 0, loaded = 0;
+  if (total > 0) copy.look(p, table, load_kt0, lo, pos + 1, p.keep);
   auto load_next = [&]() {
     if (loaded < total) {
+      if (load_item == 0) {
+        if (load_tile_no > t_begin) load_kt0 = next_kt0;
+        copy.enter();
+        if (++load_tile_no < t_end) {
+          next_kt0 = tiles.first_key(load_tile_no);
+          copy.look(p, table, next_kt0, lo, pos + 1, p.keep);
+        }
+      }
       const bool key = load_item < p.KV;
-      load_tile<HD, kDecodeThreads>(stage(loaded), key ? p.k_cache : p.v_cache, p, table, key ? load_item : c_lo + load_item - p.KV,
-                                    tiles.first_key(load_tile_no), lo, pos + 1, p.keep);
-      if (++load_item == items) { load_item = 0; ++load_tile_no; }
+      copy.load(stage(loaded), key ? p.k_cache : p.v_cache, p, table, key ? load_item : c_lo + load_item - p.KV, load_kt0, lo, pos + 1, p.keep);
+      if (++load_item == items) load_item = 0;
       ++loaded;
     }
     cp_async_commit();
   };
-  for (int n = 0; n < kDecodeStages - 1; ++n) load_next();
+  for (int n = 0; n < NS - 1; ++n) load_next();
   {  // queries: gc heads of this token, part by part; zero rows above gc
     constexpr int kChunks = HD / 8;
-    for (int i = threadIdx.x; i < p.KV * 16 * kChunks; i += kDecodeThreads) {
-      const int c = i / (16 * kChunks), qr = i / kChunks % 16, ch = i % kChunks;
+    for (int i = threadIdx.x; i < p.KV * kRows * kChunks; i += kDecodeThreads) {
+      const int c = i / (kRows * kChunks), qr = i / kChunks % kRows, ch = i % kChunks;
       uint4 v = make_uint4(0, 0, 0, 0);
       if (qr < gc) v = *reinterpret_cast<const uint4*>(p.q + (((size_t)row * p.H + head0 + qr) * p.KV + c) * HD + ch * 8);
       *reinterpret_cast<uint4*>(smem_raw + (q_tile - smem) + c * kQPart + tile_offset<HD>(qr, ch)) = v;
     }
   }
 
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float acc[HD / 8][4];
+  float m[MT][2], l[MT][2], acc[MT][HD / 8][4], s[MT][2][4];
+  uint32_t pf[MT][4];
+  int owner[MT][2];  // the value heads of a thread's two rows of each tile
 #pragma unroll
-  for (int i = 0; i < HD / 8; ++i)
+  for (int t = 0; t < MT; ++t) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-  float s[2][4];
-  uint32_t pf[4] = {0, 0, 0, 0};
+    for (int h = 0; h < 2; ++h) {
+      m[t][h] = -INFINITY;
+      l[t][h] = 0.f;
+      owner[t][h] = (head0 + t * 16 + (lane >> 2) + h * 8) / p.G;
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) pf[t][e] = 0;
+#pragma unroll
+    for (int i = 0; i < HD / 8; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[t][i][e] = 0.f;
+  }
   const int key0 = warp * 16;  // this warp's keys inside a tile
   const int krow = key0 + (lane & 7) + ((lane >> 4) << 3), kchunk = (lane >> 3) & 1;
   const int qrow = (lane & 7) + (((lane >> 3) & 1) << 3), qchunk = lane >> 4;
-  const int owner_lo = (head0 + (lane >> 2)) / p.G, owner_hi = (head0 + (lane >> 2) + 8) / p.G;  // the value heads of a thread's two rows
 
   int item = 0, kt0 = 0, tile = t_begin;
   bool live = false;
   for (int n = 0; n < total; ++n) {
-    cp_async_wait<kDecodeStages - 2>();
-    __syncthreads();  // item n has landed; everybody is done with the stage that item n + 3 takes
+    cp_async_wait<NS - 2>();
+    __syncthreads();  // item n has landed; everybody is done with the stage that the next load takes
     load_next();
     if (item == 0) {
       kt0 = tiles.first_key(tile);
       const int first = kt0 + key0;
       live = first <= pos && (first + 16 > lo || first < p.keep);  // uniform in the warp
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
+      for (int t = 0; t < MT; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[t][j][e] = 0.f;
     }
     if (live) {
       if (item < p.KV) {
         const uint32_t q_part = q_tile + (uint32_t)item * kQPart, k_tile = stage(n);
 #pragma unroll
         for (int kc = 0; kc < HD / 16; ++kc) {
-          uint32_t a[4], b[4];
-          ldmatrix_x4(a, q_part + tile_offset<HD>(qrow, kc * 2 + qchunk));
+          uint32_t b[4];
           ldmatrix_x4(b, k_tile + tile_offset<HD>(krow, kc * 2 + kchunk));
-          mma_bf16(s[0], a, b[0], b[1]);
-          mma_bf16(s[1], a, b[2], b[3]);
+#pragma unroll
+          for (int t = 0; t < MT; ++t) {
+            uint32_t a[4];
+            ldmatrix_x4(a, q_part + tile_offset<HD>(t * 16 + qrow, kc * 2 + qchunk));
+            mma_bf16(s[t][0], a, b[0], b[1]);
+            mma_bf16(s[t][1], a, b[2], b[3]);
+          }
         }
         if (item == p.KV - 1) {
 #pragma unroll
-          for (int j = 0; j < 2; ++j)
+          for (int t = 0; t < MT; ++t) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              const int key = kt0 + key0 + j * 8 + (lane & 3) * 2 + (e & 1);
-              s[j][e] = key <= pos && (key >= lo || key < p.keep) ? s[j][e] * p.scale : -INFINITY;
-            }
-          float rmax[2] = {fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1])),
-                           fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]))};
-          float corr[2], rsum[2] = {0.f, 0.f};
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 1));
-            rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 2));
-            const float m_new = fmaxf(m[h], rmax[h]);  // finite: a live warp sees at least one of its keys
-            corr[h] = __expf(m[h] - m_new);
-            m[h] = m_new;
-          }
+              for (int e = 0; e < 4; ++e) {
+                const int key = kt0 + key0 + j * 8 + (lane & 3) * 2 + (e & 1);
+                s[t][j][e] = key <= pos && (key >= lo || key < p.keep) ? s[t][j][e] * p.scale : -INFINITY;
+              }
+            float rmax[2] = {fmaxf(fmaxf(s[t][0][0], s[t][0][1]), fmaxf(s[t][1][0], s[t][1][1])),
+                             fmaxf(fmaxf(s[t][0][2], s[t][0][3]), fmaxf(s[t][1][2], s[t][1][3]))};
+            float corr[2], rsum[2] = {0.f, 0.f};
 #pragma unroll
-          for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              s[j][e] = __expf(s[j][e] - m[e >> 1]);
-              rsum[e >> 1] += s[j][e];
+            for (int h = 0; h < 2; ++h) {
+              rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 1));
+              rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 2));
+              const float m_new = fmaxf(m[t][h], rmax[h]);  // finite: a live warp sees at least one of its keys
+              corr[h] = __expf(m[t][h] - m_new);
+              m[t][h] = m_new;
             }
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 1);
-            rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 2);
-            l[h] = l[h] * corr[h] + rsum[h];
-          }
+            for (int j = 0; j < 2; ++j)
 #pragma unroll
-          for (int i = 0; i < HD / 8; ++i) {
-            acc[i][0] *= corr[0]; acc[i][1] *= corr[0];
-            acc[i][2] *= corr[1]; acc[i][3] *= corr[1];
+              for (int e = 0; e < 4; ++e) {
+                s[t][j][e] = __expf(s[t][j][e] - m[t][e >> 1]);
+                rsum[e >> 1] += s[t][j][e];
+              }
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 1);
+              rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 2);
+              l[t][h] = l[t][h] * corr[h] + rsum[h];
+            }
+#pragma unroll
+            for (int i = 0; i < HD / 8; ++i) {
+              acc[t][i][0] *= corr[0]; acc[t][i][1] *= corr[0];
+              acc[t][i][2] *= corr[1]; acc[t][i][3] *= corr[1];
+            }
+            pf[t][0] = pack_bf16(s[t][0][0], s[t][0][1]); pf[t][1] = pack_bf16(s[t][0][2], s[t][0][3]);
+            pf[t][2] = pack_bf16(s[t][1][0], s[t][1][1]); pf[t][3] = pack_bf16(s[t][1][2], s[t][1][3]);
           }
-          pf[0] = pack_bf16(s[0][0], s[0][1]); pf[1] = pack_bf16(s[0][2], s[0][3]);
-          pf[2] = pack_bf16(s[1][0], s[1][1]); pf[3] = pack_bf16(s[1][2], s[1][3]);
         }
       } else {
         const int c = c_lo + item - p.KV;  // rows of other value heads weigh nothing here
-        const uint32_t own[4] = {owner_lo == c ? pf[0] : 0u, owner_hi == c ? pf[1] : 0u, owner_lo == c ? pf[2] : 0u,
-                                 owner_hi == c ? pf[3] : 0u};
-        pv_16keys<HD>(acc, own, stage(n), key0, lane);
+        const int first_row = c * p.G - head0;
+#pragma unroll
+        for (int t = 0; t < MT; ++t) {
+          if (first_row >= (t + 1) * 16 || first_row + p.G <= t * 16) continue;  // none of this tile's rows
+          const uint32_t own[4] = {owner[t][0] == c ? pf[t][0] : 0u, owner[t][1] == c ? pf[t][1] : 0u,
+                                   owner[t][0] == c ? pf[t][2] : 0u, owner[t][1] == c ? pf[t][3] : 0u};
+          pv_16keys<HD>(acc[t], own, stage(n), key0, lane);
+        }
       }
     }
     if (++item == items) { item = 0; ++tile; }
@@ -235,20 +280,26 @@ parts_decode_kernel(const PartsParams p) {
   __syncthreads();
 
   // Merge the four warps through shared memory (over the stages): per row max, sum, acc.
-  float* mm = reinterpret_cast<float*>(smem_raw);  // [4][16]
-  float* ml = mm + 64;                             // [4][16]
-  float* ma = ml + 64;                             // [4][16][HD]
+  float* mm = reinterpret_cast<float*>(smem_raw);  // [4][kRows]
+  float* ml = mm + 4 * kRows;                      // [4][kRows]
+  float* ma = ml + 4 * kRows;                      // [4][kRows][HD]
   {
-    const int g = lane >> 2, t = lane & 3;
-    if (t == 0) {
-      mm[warp * 16 + g] = m[0]; mm[warp * 16 + g + 8] = m[1];
-      ml[warp * 16 + g] = l[0]; ml[warp * 16 + g + 8] = l[1];
-    }
+    const int g = lane >> 2, q = lane & 3;
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) {
-      if (g < gc) *reinterpret_cast<float2*>(ma + ((size_t)(warp * 16 + g) * HD + i * 8 + t * 2)) = make_float2(acc[i][0], acc[i][1]);
-      if (g + 8 < gc) *reinterpret_cast<float2*>(ma + ((size_t)(warp * 16 + g + 8) * HD + i * 8 + t * 2)) = make_float2(acc[i][2], acc[i][3]);
-    }
+    for (int t = 0; t < MT; ++t)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int rr = t * 16 + h * 8 + g, at = warp * kRows + rr;
+        if (q == 0) {
+          mm[at] = m[t][h];
+          ml[at] = l[t][h];
+        }
+        if (rr < gc) {
+#pragma unroll
+          for (int i = 0; i < HD / 8; ++i)
+            *reinterpret_cast<float2*>(ma + (size_t)at * HD + i * 8 + q * 2) = make_float2(acc[t][i][2 * h], acc[t][i][2 * h + 1]);
+        }
+      }
   }
   __syncthreads();
   for (int i = threadIdx.x; i < gc * HD; i += kDecodeThreads) {
@@ -256,14 +307,14 @@ parts_decode_kernel(const PartsParams p) {
     float mx = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w)
-      if (ml[w * 16 + qr] > 0.f) mx = fmaxf(mx, mm[w * 16 + qr]);
+      if (ml[w * kRows + qr] > 0.f) mx = fmaxf(mx, mm[w * kRows + qr]);
     float a = 0.f, den = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w)
-      if (ml[w * 16 + qr] > 0.f) {
-        const float f = __expf(mm[w * 16 + qr] - mx);
-        den += ml[w * 16 + qr] * f;
-        a += ma[(size_t)(w * 16 + qr) * HD + col] * f;
+      if (ml[w * kRows + qr] > 0.f) {
+        const float f = __expf(mm[w * kRows + qr] - mx);
+        den += ml[w * kRows + qr] * f;
+        a += ma[(size_t)(w * kRows + qr) * HD + col] * f;
       }
     if (p.NP == 1) {
       p.out[((size_t)row * p.H + head0 + qr) * HD + col] = __float2bfloat16_rn(a / den);
@@ -326,14 +377,23 @@ parts_prefill_kernel(const PartsParams p) {
       cp_async16(at + tile_offset<HD>(rr, ch), p.q + (((size_t)(row0 + qi) * p.H + head0 + g) * p.KV + c) * HD + ch * 8, real);
     }
   };
-  int load_tile_no = 0, load_item = 0, loaded = 0;
+  TileCopy<HD, kPrefillThreads> copy(p);
+  int load_kt0 = tiles.first_key(0), next_kt0 = 0, load_tile_no = 0, load_item = 0, loaded = 0;
+  copy.look(p, table, load_kt0, lo, hi, p.keep);
   auto load_next = [&]() {
     if (loaded < total) {
+      if (load_item == 0) {
+        if (load_tile_no > 0) load_kt0 = next_kt0;
+        copy.enter();
+        if (++load_tile_no < tiles.count) {
+          next_kt0 = tiles.first_key(load_tile_no);
+          copy.look(p, table, next_kt0, lo, hi, p.keep);
+        }
+      }
       const bool key = load_item < p.KV;
-      load_tile<HD, kPrefillThreads>(stage(loaded), key ? p.k_cache : p.v_cache, p, table, key ? load_item : kvh,
-                                     tiles.first_key(load_tile_no), lo, hi, p.keep);
+      copy.load(stage(loaded), key ? p.k_cache : p.v_cache, p, table, key ? load_item : kvh, load_kt0, lo, hi, p.keep);
       if (kStreamQ && key) load_queries(stage(loaded) + kTileBytes, load_item);
-      if (++load_item == items) { load_item = 0; ++load_tile_no; }
+      if (++load_item == items) load_item = 0;
       ++loaded;
     }
     cp_async_commit();
@@ -461,7 +521,19 @@ parts_prefill_kernel(const PartsParams p) {
 
 constexpr size_t kMaxSmem = 227 * 1024;
 
-size_t decode_smem(int hd, int KV) { return (size_t)kDecodeStages * kKeyTile * hd * 2 + (size_t)KV * 16 * hd * 2; }
+int decode_tiles(int H) { return H > 16 ? 2 : 1; }
+size_t decode_smem(int hd, int H, int KV, int stages) {
+  return (size_t)stages * kKeyTile * hd * 2 + (size_t)KV * decode_tiles(H) * 16 * hd * 2;
+}
+// four stages where two blocks then share an SM, else eight where they fit (one block keeps the copies going)
+int decode_stages(int hd, int H, int KV) {
+  return decode_smem(hd, H, KV, 4) > 113 * 1024 && decode_smem(hd, H, KV, 8) <= kMaxSmem ? 8 : 4;
+}
+// heads per block: whole groups where they fit its rows, so that no value head is read twice
+int decode_heads(int H, int KV) {
+  const int G = H / KV, most = 16 * decode_tiles(H);
+  return H <= most ? H : (G <= most ? most / G * G : most);
+}
 size_t prefill_smem(int hd, int KV, bool stream) {
   const size_t tile = (size_t)kKeyTile * hd * 2, q = (size_t)kPrefillRows * hd * 2;
   return stream ? kPrefillStages * (tile + q) : kPrefillStages * tile + KV * q;
@@ -475,15 +547,25 @@ int start(Kernel kern, dim3 grid, int threads, size_t smem, cudaStream_t stream,
   return asb::check_launch(what);
 }
 
+template <typename F>
+auto with_decode_kernel(int hd, int H, int KV, F&& use) {
+  const bool two = decode_tiles(H) == 2, eight = decode_stages(hd, H, KV) == 8;
+#define ASB_PICK(HD) \
+  (two ? (eight ? use(parts_decode_kernel<HD, 2, 8>) : use(parts_decode_kernel<HD, 2, 4>)) \
+       : (eight ? use(parts_decode_kernel<HD, 1, 8>) : use(parts_decode_kernel<HD, 1, 4>)))
+  return hd == 64 ? ASB_PICK(64) : ASB_PICK(128);
+#undef ASB_PICK
+}
+
 template <int HD>
 int launch_parts(PartsParams p, int run_decode, int run_prefill, cudaStream_t stream) {
   if (run_decode) {
-    // whole groups of heads per block where they fit 16 rows, so that no value head is read twice
-    p.GC = p.H <= 16 ? p.H : (p.G <= 16 ? 16 / p.G * p.G : 16);
+    p.GC = decode_heads(p.H, p.KV);
     p.HC = (p.H + p.GC - 1) / p.GC;
     if (p.HC > 65535) return asb::fail("attention_parts: too many heads");
     dim3 grid(p.short_rows > 0 ? p.short_rows : p.T, p.HC, p.NP);
-    if (int rc = start(parts_decode_kernel<HD>, grid, kDecodeThreads, decode_smem(HD, p.KV), stream, p, "parts_decode")) return rc;
+    const size_t smem = decode_smem(HD, p.H, p.KV, decode_stages(HD, p.H, p.KV));
+    if (int rc = with_decode_kernel(HD, p.H, p.KV, [&](auto kern) { return start(kern, grid, kDecodeThreads, smem, stream, p, "parts_decode"); })) return rc;
   }
   if (run_prefill) {
     p.GC = p.G < 16 ? p.G : 16;
@@ -502,28 +584,23 @@ int launch_parts(PartsParams p, int run_decode, int run_prefill, cudaStream_t st
 
 }  // namespace
 
-// 1 if these kernels serve (head size, kv heads): the decode kernel keeps a token's queries of all parts
-// in shared memory.
-extern "C" int asb_attention_parts_supported(int hd, int KV) {
-  return (hd == 64 || hd == 128) && KV >= 1 && decode_smem(hd, KV) <= kMaxSmem ? 1 : 0;
+// 1 if these kernels serve the shape: the decode kernel keeps a token's queries of all parts in shared memory.
+extern "C" int asb_attention_parts_supported(int hd, int H, int KV) {
+  return (hd == 64 || hd == 128) && KV >= 1 && decode_smem(hd, H, KV, 4) <= kMaxSmem ? 1 : 0;
 }
 
 // Query heads that share a block of the decode kernel, and blocks the device holds at once: for the
 // caller's choice of partitions.
-extern "C" int asb_attention_parts_heads(int H, int KV) {
-  const int G = H / KV;
-  return H <= 16 ? H : (G <= 16 ? 16 / G * G : 16);
-}
-extern "C" int asb_attention_parts_resident(int hd, int KV) {
-  if (!asb_attention_parts_supported(hd, KV)) return 0;
+extern "C" int asb_attention_parts_heads(int H, int KV) { return decode_heads(H, KV); }
+extern "C" int asb_attention_parts_resident(int hd, int H, int KV) {
+  if (!asb_attention_parts_supported(hd, H, KV)) return 0;
   int device = 0, sms = 0, per_sm = 0;
   if (cudaGetDevice(&device) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess) return 0;
-  const size_t smem = decode_smem(hd, KV);
-  auto ask = [&](auto kern) {
+  const size_t smem = decode_smem(hd, H, KV, decode_stages(hd, H, KV));
+  const cudaError_t e = with_decode_kernel(hd, H, KV, [&](auto kern) {
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kern, kDecodeThreads, smem);
-  };
-  const cudaError_t e = hd == 64 ? ask(parts_decode_kernel<64>) : ask(parts_decode_kernel<128>);
+  });
   return e == cudaSuccess ? per_sm * sms : 0;
 }
 
@@ -538,7 +615,7 @@ extern "C" int asb_attention_parts(void* out, const void* q, const void* k_cache
                                    int run_decode, int run_prefill, int all_single, int short_rows, cudaStream_t stream) {
   if (num_tokens == 0 || R == 0) return 0;
   if (KV < 1 || H % KV) return asb::fail("attention_parts: %d heads over %d kv heads", H, KV);
-  if (!asb_attention_parts_supported(hd, KV)) return asb::fail("attention_parts: head_dim %d with %d key heads is not served", hd, KV);
+  if (!asb_attention_parts_supported(hd, H, KV)) return asb::fail("attention_parts: head_dim %d with %d key heads is not served", hd, KV);
   if (window < 0 || keep < 0 || bs < 1) return asb::fail("attention_parts: window %d, keep %d, page %d", window, keep, bs);
   if (NP < 1 || NP > 65535 || PT < 1) return asb::fail("attention_parts: %d partitions of %d tiles", NP, PT);
   if (NP > 1 && (!part_m || !part_l || !part_acc)) return asb::fail("attention_parts: %d partitions need scratch", NP);

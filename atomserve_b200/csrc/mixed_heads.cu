@@ -46,16 +46,35 @@ struct MixedParams {
   float eps, lambda;
 };
 
+template <typename T>
+__device__ __forceinline__ void store4(T* at, const float (&v)[4]) {
+  if constexpr (sizeof(T) == 2) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(at) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+  } else {
+    *reinterpret_cast<float4*>(at) = make_float4(v[0], v[1], v[2], v[3]);
+  }
+}
+template <typename T>
+__device__ __forceinline__ void load4(const T* at, float (&v)[4]) {
+  if constexpr (sizeof(T) == 2) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(at);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  } else {
+    const float4 f = *reinterpret_cast<const float4*>(at);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  }
+}
+
 // V neighbouring columns of a token's projection, bias added
 template <typename T, int V>
-__device__ __forceinline__ void column(const MixedParams& p, int t, int col, float (&v)[V]) {
+__device__ __forceinline__ void column(const MixedParams& p, int t, int col, float (&v)[V], bool biased = true) {
   if (p.proj) {
     const T* at = (const T*)p.proj + (size_t)t * p.row + col;
-    if constexpr (V == 4 && sizeof(T) == 2) {
-      const uint2 raw = *reinterpret_cast<const uint2*>(at);
-      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-      v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+    if constexpr (V == 4) {
+      load4<T>(at, v);
     } else {
 #pragma unroll
       for (int k = 0; k < V; ++k) v[k] = asb::to_float(at[k]);
@@ -63,7 +82,7 @@ __device__ __forceinline__ void column(const MixedParams& p, int t, int col, flo
   } else {
     asb::partial_sum<V>(p.ps, t, col, asb::partial_slots(p.ps, col / asb::kPartialRows), v);
   }
-  if (p.bias) {
+  if (biased && p.bias) {
 #pragma unroll
     for (int k = 0; k < V; ++k) v[k] += p.bias[col + k];
   }
@@ -122,10 +141,8 @@ __device__ __forceinline__ void norm_and_turn(const MixedParams& p, float* x, in
   }
 }
 
-// One block per token. V: columns read at a time. R: query heads per kv head whose queries a thread
-// holds in registers (8 entries of each) while it walks the output heads; 0: any number, read from
-// shared memory as they are needed.
-template <typename T, int V, int R>
+// The general form: any sizes, both pairings. One block per token; V: columns read at a time.
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 mixed_heads_prepare_kernel(const MixedParams p) {
   extern __shared__ __align__(16) float smem[];
@@ -189,80 +206,193 @@ mixed_heads_prepare_kernel(const MixedParams p) {
   }
   __syncthreads();
   T* q_out = (T*)p.q_out + (size_t)t * H * KV * hd;
-  if constexpr (R > 0) {
-    const int per = hd >> 3;  // (8 divides hd; R is the group size)
-    if (store)
-      for (int i = threadIdx.x; i < KV * per; i += blockDim.x) {
-        const int c = i / per, e = (i - c * per) << 3;
-        float v[8];
-#pragma unroll
-        for (int k = 0; k < 8; ++k) v[k] = k_s[c * hd + e + k];
-        store8<T>((T*)p.k_cache + ((page * KV + c) * p.bs + off) * hd + e, v);
-      }
-    // (part, 8 entries) per thread; the threads that are left over share the output heads
-    const int items = KV * per, lanes = items < (int)blockDim.x ? (int)blockDim.x / items : 1;
-    for (int item = threadIdx.x % items + (threadIdx.x / items >= lanes ? items : 0), first = threadIdx.x / items; item < items;
-         item += blockDim.x) {
-      const int c = item / per, e = (item - c * per) << 3;
-      float q[R][8];
-#pragma unroll
-      for (int g = 0; g < R; ++g) {
-        const float4 a = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e);
-        const float4 b = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e + 4);
-        q[g][0] = a.x; q[g][1] = a.y; q[g][2] = a.z; q[g][3] = a.w;
-        q[g][4] = b.x; q[g][5] = b.y; q[g][6] = b.z; q[g][7] = b.w;
-      }
-      for (int h = items < (int)blockDim.x ? first : 0; h < H; h += lanes) {
-        float v[8];
-#pragma unroll
-        for (int k = 0; k < 8; ++k) v[k] = 0.f;
-#pragma unroll
-        for (int g = 0; g < R; ++g) {
-          const float w = talk_s[h * H + c * R + g];
-#pragma unroll
-          for (int k = 0; k < 8; ++k) v[k] = fmaf(w, q[g][k], v[k]);
-        }
-        store8<T>(q_out + ((size_t)h * KV + c) * hd + e, v);
-      }
+  if (store)
+    for (int i = threadIdx.x; i < KV * hd; i += blockDim.x) {
+      const int c = i / hd, e = i - c * hd;
+      ((T*)p.k_cache)[((page * KV + c) * p.bs + off) * hd + e] = asb::from_float<T>(k_s[i]);
     }
-  } else {
-    if (store)
-      for (int i = threadIdx.x; i < KV * hd; i += blockDim.x) {
-        const int c = i / hd, e = i - c * hd;
-        ((T*)p.k_cache)[((page * KV + c) * p.bs + off) * hd + e] = asb::from_float<T>(k_s[i]);
+  for (int i = threadIdx.x; i < H * KV * hd; i += blockDim.x) {
+    const int e = i % hd, hc = i / hd, c = hc % KV, h = hc / KV;
+    float v = 0.f;
+    for (int g = c * G; g < (c + 1) * G; ++g) v = fmaf(talk_s[h * H + g], q_s[g * hd + e], v);
+    q_out[i] = asb::from_float<T>(v);
+  }
+}
+
+// The usual form: neighbouring pairs (or no rotation), head sizes that are multiples of 8. A thread keeps
+// its vectors of four columns in registers from the projection to where they belong: both entries of a
+// pair lie in one vector, so norm and rotation touch no shared memory; keys and values go to their
+// pages and queries to shared memory for the mix. kPer: vectors a thread. R and E: the group's heads
+// whose E entries a thread holds while it walks the output heads.
+template <typename T, int R, int E, int kPer>
+__global__ void __launch_bounds__(256, kPer <= 4 ? 3 : 2)
+mixed_heads_prepare_vec_kernel(const MixedParams p) {
+  extern __shared__ __align__(16) float smem[];
+  __shared__ float scratch[2][8];
+  const int H = p.H, KV = p.KV, hd = p.hd, dim = p.dim;
+  float* q_s = smem;              // [H][hd], zeros behind dim
+  float* talk_s = q_s + H * hd;   // [H][H]
+  float* cs = talk_s + H * H;     // [rotary_dim] cosines, then sines
+  const int nq = H * dim >> 2, nk = KV * dim >> 2, nv = p.k_cache ? KV * p.vdim >> 2 : 0, total = nq + (p.k_cache ? nk + nv : 0);
+  // what no kernel writes is read before the wait
+  for (int i = threadIdx.x; i < H * H; i += 256) talk_s[i] = p.talk[i];
+  for (int i = threadIdx.x; i < H * (hd - dim); i += 256) q_s[i / (hd - dim) * hd + dim + i % (hd - dim)] = 0.f;
+  float4 bias[kPer], gain[kPer];
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    bias[u] = p.bias && i < total ? *reinterpret_cast<const float4*>(p.bias + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    gain[u] = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (p.q_gain && i < nq) gain[u] = *reinterpret_cast<const float4*>(p.q_gain + 4 * i);
+    else if (p.q_gain && i < nq + nk) gain[u] = *reinterpret_cast<const float4*>(p.k_gain + 4 * (i - nq));
+  }
+  asb::pdl_wait();
+  asb::pdl_launch_dependents();
+  const int t = blockIdx.x, half = p.rotary_dim >> 1;
+  float v[kPer][4];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    if (i < total) column<T, 4>(p, t, 4 * i, v[u], false);
+  }
+  const float position = (float)__ldcg(p.positions + t);
+  for (int i = threadIdx.x; i < half; i += 256) sincosf(position * p.inv_freq[i], &cs[half + i], &cs[i]);
+  const int slot = p.slots ? __ldcg(p.slots + t) : -1;
+  const bool store = p.k_cache && slot >= 0;
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    if (i >= total) continue;
+    v[u][0] += bias[u].x; v[u][1] += bias[u].y; v[u][2] += bias[u].z; v[u][3] += bias[u].w;
+    const float ss = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
+    if (i < nq) sq += ss;
+    else if (i < nq + nk) sk += ss;
+  }
+  sq = asb::warp_sum(sq);
+  sk = asb::warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    scratch[0][threadIdx.x >> 5] = sq;
+    scratch[1][threadIdx.x >> 5] = sk;
+  }
+  __syncthreads();  // (the angles too)
+  float inv_q = 1.f, inv_k = 1.f;
+  if (p.q_gain) {
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      sq += scratch[0][w];
+      sk += scratch[1][w];
+    }
+    inv_q = 1.f / sqrtf(sq / (float)(H * dim) + p.eps);
+    inv_k = 1.f / sqrtf(sk / (float)(KV * dim) + p.eps);
+  }
+  const size_t page = store ? slot / p.bs : 0, off = store ? slot % p.bs : 0;
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    if (i >= total) continue;
+    if (i < nq + nk) {
+      const bool query = i < nq;
+      const int col = 4 * (query ? i : i - nq), h = col / dim, e = col - h * dim;
+      const float inv = query ? inv_q : inv_k;
+      const float g[4] = {gain[u].x, gain[u].y, gain[u].z, gain[u].w};
+      float w[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) w[k] = v[u][k] * inv * g[k];
+#pragma unroll
+      for (int k = 0; k < 4; k += 2) {
+        const int pair = (e + k) >> 1;
+        if (pair < half) {
+          const float c = cs[pair], s = cs[half + pair], a = w[k], b = w[k + 1];
+          w[k] = a * c - b * s;
+          w[k + 1] = b * c + a * s;
+        }
       }
-    for (int i = threadIdx.x; i < H * KV * hd; i += blockDim.x) {
-      const int e = i % hd, hc = i / hd, c = hc % KV, h = hc / KV;
-      float v = 0.f;
-      for (int g = c * G; g < (c + 1) * G; ++g) v = fmaf(talk_s[h * H + g], q_s[g * hd + e], v);
-      q_out[i] = asb::from_float<T>(v);
+      if (query) *reinterpret_cast<float4*>(q_s + h * hd + e) = make_float4(w[0], w[1], w[2], w[3]);
+      else if (store) store4<T>((T*)p.k_cache + ((page * KV + h) * p.bs + off) * hd + e, w);
+    } else {
+      const int col = 4 * (i - nq - nk), h = col / p.vdim, e = col - h * p.vdim;
+      const size_t at = (size_t)t * KV * p.vdim + col;
+      if (p.v_out) store4<T>((T*)p.v_out + at, v[u]);
+      if (p.v_first) {
+        float f[4];
+        load4<T>((const T*)p.v_first + at, f);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[u][k] = (1.f - p.lambda) * v[u][k] + p.lambda * f[k];
+      }
+      if (store) store4<T>((T*)p.v_cache + ((page * KV + h) * p.bs + off) * hd + e, v[u]);
+    }
+  }
+  if (store) {  // zeros behind what a head holds
+    const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+    const int kz = (hd - dim) >> 2, vz = (hd - p.vdim) >> 2;
+    for (int i = threadIdx.x; i < KV * kz; i += 256) store4<T>((T*)p.k_cache + ((page * KV + i / kz) * p.bs + off) * hd + dim + i % kz * 4, zero);
+    for (int i = threadIdx.x; i < KV * vz; i += 256) store4<T>((T*)p.v_cache + ((page * KV + i / vz) * p.bs + off) * hd + p.vdim + i % vz * 4, zero);
+  }
+  __syncthreads();
+  T* q_out = (T*)p.q_out + (size_t)t * H * KV * hd;
+  // (part, E entries) per thread; the threads that are left over share the output heads
+  const int per = hd / E, items = KV * per, lanes = items < 256 ? 256 / items : 1;
+  if ((int)threadIdx.x >= items * lanes) return;
+  for (int item = threadIdx.x % items; item < items; item += 256) {
+    const int c = item / per, e = (item - c * per) * E;
+    float q[R][E];
+#pragma unroll
+    for (int g = 0; g < R; ++g)
+#pragma unroll
+      for (int k = 0; k < E; k += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e + k);
+        q[g][k] = f.x; q[g][k + 1] = f.y; q[g][k + 2] = f.z; q[g][k + 3] = f.w;
+      }
+    for (int h = items < 256 ? threadIdx.x / items : 0; h < H; h += lanes) {
+      float sum[E], w[R];
+#pragma unroll
+      for (int g = 0; g < R; ++g) w[g] = talk_s[h * H + c * R + g];
+#pragma unroll
+      for (int k = 0; k < E; ++k) sum[k] = 0.f;
+#pragma unroll
+      for (int g = 0; g < R; ++g)
+#pragma unroll
+        for (int k = 0; k < E; ++k) sum[k] = fmaf(w[g], q[g][k], sum[k]);
+      T* at = q_out + ((size_t)h * KV + c) * hd + e;
+      if constexpr (E == 8) store8<T>(at, sum);
+      else store4<T>(at, sum);
     }
   }
 }
 
-template <typename T, int V, int R>
-int run(const MixedParams& p, int tokens, size_t smem, cudaStream_t stream) {
-  auto kern = mixed_heads_prepare_kernel<T, V, R>;
+template <typename T, typename Kernel>
+int start(Kernel kern, const MixedParams& p, int tokens, size_t smem, cudaStream_t stream) {
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return asb::fail("mixed_heads_prepare: shared memory %zu: %s", smem, cudaGetErrorString(e));
   asb::launch(kern, tokens, 256, smem, stream, p);
   return asb::check_launch("mixed_heads_prepare");
 }
 
+template <typename T, int R, int E>
+int start_vec(const MixedParams& p, int tokens, int vectors, size_t smem, cudaStream_t stream) {
+  if (vectors <= 2 * 256) return start<T>(mixed_heads_prepare_vec_kernel<T, R, E, 2>, p, tokens, smem, stream);
+  if (vectors <= 4 * 256) return start<T>(mixed_heads_prepare_vec_kernel<T, R, E, 4>, p, tokens, smem, stream);
+  return start<T>(mixed_heads_prepare_vec_kernel<T, R, E, 8>, p, tokens, smem, stream);
+}
+
 template <typename T>
 int dispatch(const MixedParams& p, int tokens, cudaStream_t stream) {
   const size_t smem = sizeof(float) * ((size_t)(p.H + p.KV) * p.hd + (size_t)p.H * p.H + p.rotary_dim + 4);
   if (smem > 220 * 1024) return asb::fail("mixed_heads_prepare: %d heads of %d need %zu bytes of shared memory", p.H, p.hd, smem);
-  const int G = p.H / p.KV;
+  const int G = p.H / p.KV, vectors = (p.H * p.dim + p.KV * (p.dim + p.vdim)) / 4;
   const bool four = p.dim % 4 == 0 && p.vdim % 4 == 0 && p.row % 4 == 0 &&
                     (((uintptr_t)p.proj | (uintptr_t)p.ps.ws) & 15) == 0;
-  const bool eight = four && p.hd % 8 == 0 && (((uintptr_t)p.q_out | (uintptr_t)p.k_cache) & 15) == 0;
-  if (eight && G == 1) return run<T, 4, 1>(p, tokens, smem, stream);
-  if (eight && G == 2) return run<T, 4, 2>(p, tokens, smem, stream);
-  if (eight && G == 4) return run<T, 4, 4>(p, tokens, smem, stream);
-  if (eight && G == 8) return run<T, 4, 8>(p, tokens, smem, stream);
-  if (four) return run<T, 4, 0>(p, tokens, smem, stream);
-  return run<T, 1, 0>(p, tokens, smem, stream);
+  const bool eight = four && p.hd % 8 == 0 && vectors <= 8 * 256 && (p.interleaved || p.rotary_dim == 0) &&
+                     (((uintptr_t)p.q_out | (uintptr_t)p.k_cache | (uintptr_t)p.v_cache | (uintptr_t)p.v_first | (uintptr_t)p.v_out |
+                       (uintptr_t)p.bias | (uintptr_t)p.q_gain | (uintptr_t)p.k_gain) & 15) == 0;
+  if (eight && G == 1) return start_vec<T, 1, 8>(p, tokens, vectors, smem, stream);
+  if (eight && G == 2) return start_vec<T, 2, 8>(p, tokens, vectors, smem, stream);
+  if (eight && G == 4) return start_vec<T, 4, 8>(p, tokens, vectors, smem, stream);
+  if (eight && G == 8) return start_vec<T, 8, 4>(p, tokens, vectors, smem, stream);
+  if (four) return start<T>(mixed_heads_prepare_kernel<T, 4>, p, tokens, smem, stream);
+  return start<T>(mixed_heads_prepare_kernel<T, 1>, p, tokens, smem, stream);
 }
 
 }  // namespace

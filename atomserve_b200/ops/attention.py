@@ -166,7 +166,7 @@ def paged_attention(
     if q.dtype == torch.bfloat16 and not generic and not summed and not keep and lib().asb_attention_mma_supported(hd, H // KV):
         return _paged_attention_mma(q, out, k_cache, v_cache, block_tables, req_q_start, req_pos_start,
                                     num_requests, max_context, win, scale, partitions, host_q_lens, sink, chunk, softcap, span)  # fmt: skip
-    if q.dtype == torch.bfloat16 and not generic and summed and not chunk and not softcap and sink is None and lib().asb_attention_parts_supported(hd, KV):
+    if q.dtype == torch.bfloat16 and not generic and summed and not chunk and not softcap and sink is None and lib().asb_attention_parts_supported(hd, H, KV):
         return _paged_attention_parts(q, out, k_cache, v_cache, block_tables, req_q_start, req_pos_start, num_requests, max_context,
                                       win, keep, scale, partitions, host_q_lens)  # fmt: skip
     ps, np_ = partitions or plan_partitions(T, num_requests, KV, H // KV, max_context, span)
@@ -278,11 +278,11 @@ def _paged_attention_mma(q, out, k_cache, v_cache, block_tables, req_q_start, re
 @functools.lru_cache(maxsize=4096)
 def plan_parts_partitions(rows: int, heads: int, kv_heads: int, max_context: int, window: int, keep: int, head_dim: int) -> tuple[int, int]:
     """(key tiles of 64 per partition, partitions) for the decode kernel of heads with a vector per
-    key head, one block per (row, up to 16 heads, partition): the same weighing as
+    key head, one block per (row, up to 32 heads, partition): the same weighing as
     `plan_decode_partitions`, a tile's cost being the key and value heads that the block walks."""
     per_block = lib().asb_attention_parts_heads(heads, kv_heads)
     chunks = -(-heads // per_block)
-    resident = lib().asb_attention_parts_resident(head_dim, kv_heads) or 148
+    resident = lib().asb_attention_parts_resident(head_dim, heads, kv_heads) or 148
     tiles = -(-max_context // 64)
     if window:
         tiles = min(tiles, -(-min(keep, max_context) // 64) + -(-window // 64) + 1)

@@ -115,9 +115,9 @@ _SIGNATURES = {
     "asb_attention_parts": [_P] * 10 + [_I] * 11 + [_F] + [_I] * 4 + [_P],
     "asb_attention_parts_tcgen05": [_P] * 7 + [_I] * 10 + [_F, _P, _P],
     "asb_attention_parts_tcgen05_supported": [_I, _I, _I],
-    "asb_attention_parts_supported": [_I, _I],
+    "asb_attention_parts_supported": [_I, _I, _I],
     "asb_attention_parts_heads": [_I, _I],
-    "asb_attention_parts_resident": [_I, _I],
+    "asb_attention_parts_resident": [_I, _I, _I],
     "asb_moe_relu2": [_P] * 5 + [_I] * 5 + [_P],
     "asb_moe_relu2_mma": [_P] * 5 + [_I] * 4 + [_P],
     # heads of several score maps
