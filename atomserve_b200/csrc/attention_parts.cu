@@ -7,8 +7,8 @@
 //   decode   one block per (new token, up to 32 query heads, key partition): the heads are the rows
 //            of one or two 16-row tiles, so a key is read once for all of them. Per tile of 64 keys the block
 //            walks the KV key heads, the scores growing in registers, and then the value heads that
-//            its rows belong to, each with the other rows' weights at zero. Four warps share a tile,
-//            sixteen keys apiece, and merge at the end. Serves requests of at most kShortRows tokens.
+//            its rows belong to, each with the other rows' weights at zero. Four warps per row tile
+//            share the keys, sixteen apiece, and merge at the end. Serves requests of at most kShortRows tokens.
 //   prefill  one block per (request, tile of tokens, kv head): 128 rows = (token, head) pairs, sixteen
 //            per warp; per tile of 64 keys the KV key heads, then the kv head's values. The queries
 //            of all parts stay in shared memory where they fit; otherwise a part's queries come with
@@ -28,7 +28,6 @@ using namespace asb::mma;
 
 constexpr int kKeyTile = 64;
 constexpr int kShortRows = 8;  // requests with at most this many new tokens go row by row
-constexpr int kDecodeThreads = 128;
 constexpr int kPrefillThreads = 256, kPrefillRows = 128;
 
 struct PartsParams {
@@ -101,14 +100,15 @@ struct TileCopy {
 
 // ---- decode ------------------------------------------------------------------------------------
 
-// MT: tiles of 16 query heads; NS: stages of the ring
-template <int HD, int MT, int NS>
-__global__ void __launch_bounds__(kDecodeThreads)
+// WG: groups of four warps, each with 16 query heads of its own and all of a tile's keys; NS: stages of
+// the ring (with four, two blocks share an SM)
+template <int HD, int WG, int NS>
+__global__ void __launch_bounds__(128 * WG, NS == 4 ? 2 : 1)
 parts_decode_kernel(const PartsParams p) {
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   extern __shared__ __align__(128) unsigned char smem_raw[];
-  constexpr int kTileBytes = kKeyTile * HD * 2, kRows = 16 * MT, kQPart = kRows * HD * 2;
+  constexpr int kTileBytes = kKeyTile * HD * 2, kThreads = 128 * WG, kRows = 16 * WG, kQPart = kRows * HD * 2;
   const uint32_t smem = smem_u32(smem_raw);
   auto stage = [&](int n) { return smem + (uint32_t)(n % NS) * kTileBytes; };
   const uint32_t q_tile = smem + NS * kTileBytes;  // [KV][kRows]
@@ -134,7 +134,7 @@ parts_decode_kernel(const PartsParams p) {
   const int t_begin = blockIdx.z * p.PT, t_end = min(tiles.count, t_begin + p.PT);
   const int total = max(0, t_end - t_begin) * items;
 
-  TileCopy<HD, kDecodeThreads> copy(p);
+  TileCopy<HD, kThreads> copy(p);
   int load_kt0 = tiles.first_key(t_begin), next_kt0 = 0, load_tile_no = t_begin, load_item = 0, loaded = 0;
   if (total > 0) copy.look(p, table, load_kt0, lo, pos + 1, p.keep);
   auto load_next = [&]() {
@@ -157,7 +157,7 @@ parts_decode_kernel(const PartsParams p) {
   for (int n = 0; n < NS - 1; ++n) load_next();
   {  // queries: gc heads of this token, part by part; zero rows above gc
     constexpr int kChunks = HD / 8;
-    for (int i = threadIdx.x; i < p.KV * kRows * kChunks; i += kDecodeThreads) {
+    for (int i = threadIdx.x; i < p.KV * kRows * kChunks; i += kThreads) {
       const int c = i / (kRows * kChunks), qr = i / kChunks % kRows, ch = i % kChunks;
       uint4 v = make_uint4(0, 0, 0, 0);
       if (qr < gc) v = *reinterpret_cast<const uint4*>(p.q + (((size_t)row * p.H + head0 + qr) * p.KV + c) * HD + ch * 8);
@@ -165,27 +165,23 @@ parts_decode_kernel(const PartsParams p) {
     }
   }
 
-  float m[MT][2], l[MT][2], acc[MT][HD / 8][4], s[MT][2][4];
-  uint32_t pf[MT][4];
-  int owner[MT][2];  // the value heads of a thread's two rows of each tile
+  float m[2], l[2], acc[HD / 8][4], s[2][4];
+  uint32_t pf[4] = {0, 0, 0, 0};
+  const int group = warp >> 2;         // this warp's 16 heads
+  const int key0 = (warp & 3) * 16;    // and its keys inside a tile
+  int owner[2];                        // the value heads of a thread's two rows
 #pragma unroll
-  for (int t = 0; t < MT; ++t) {
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      m[t][h] = -INFINITY;
-      l[t][h] = 0.f;
-      owner[t][h] = (head0 + t * 16 + (lane >> 2) + h * 8) / p.G;
-    }
-#pragma unroll
-    for (int e = 0; e < 4; ++e) pf[t][e] = 0;
-#pragma unroll
-    for (int i = 0; i < HD / 8; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[t][i][e] = 0.f;
+  for (int h = 0; h < 2; ++h) {
+    m[h] = -INFINITY;
+    l[h] = 0.f;
+    owner[h] = (head0 + group * 16 + (lane >> 2) + h * 8) / p.G;
   }
-  const int key0 = warp * 16;  // this warp's keys inside a tile
+#pragma unroll
+  for (int i = 0; i < HD / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
   const int krow = key0 + (lane & 7) + ((lane >> 4) << 3), kchunk = (lane >> 3) & 1;
-  const int qrow = (lane & 7) + (((lane >> 3) & 1) << 3), qchunk = lane >> 4;
+  const int qrow = group * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), qchunk = lane >> 4;
 
   int item = 0, kt0 = 0, tile = t_begin;
   bool live = false;
@@ -198,80 +194,67 @@ parts_decode_kernel(const PartsParams p) {
       const int first = kt0 + key0;
       live = first <= pos && (first + 16 > lo || first < p.keep);  // uniform in the warp
 #pragma unroll
-      for (int t = 0; t < MT; ++t)
+      for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[t][j][e] = 0.f;
+        for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
     }
     if (live) {
       if (item < p.KV) {
         const uint32_t q_part = q_tile + (uint32_t)item * kQPart, k_tile = stage(n);
 #pragma unroll
         for (int kc = 0; kc < HD / 16; ++kc) {
-          uint32_t b[4];
+          uint32_t a[4], b[4];
+          ldmatrix_x4(a, q_part + tile_offset<HD>(qrow, kc * 2 + qchunk));
           ldmatrix_x4(b, k_tile + tile_offset<HD>(krow, kc * 2 + kchunk));
-#pragma unroll
-          for (int t = 0; t < MT; ++t) {
-            uint32_t a[4];
-            ldmatrix_x4(a, q_part + tile_offset<HD>(t * 16 + qrow, kc * 2 + qchunk));
-            mma_bf16(s[t][0], a, b[0], b[1]);
-            mma_bf16(s[t][1], a, b[2], b[3]);
-          }
+          mma_bf16(s[0], a, b[0], b[1]);
+          mma_bf16(s[1], a, b[2], b[3]);
         }
         if (item == p.KV - 1) {
 #pragma unroll
-          for (int t = 0; t < MT; ++t) {
+          for (int j = 0; j < 2; ++j)
 #pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                const int key = kt0 + key0 + j * 8 + (lane & 3) * 2 + (e & 1);
-                s[t][j][e] = key <= pos && (key >= lo || key < p.keep) ? s[t][j][e] * p.scale : -INFINITY;
-              }
-            float rmax[2] = {fmaxf(fmaxf(s[t][0][0], s[t][0][1]), fmaxf(s[t][1][0], s[t][1][1])),
-                             fmaxf(fmaxf(s[t][0][2], s[t][0][3]), fmaxf(s[t][1][2], s[t][1][3]))};
-            float corr[2], rsum[2] = {0.f, 0.f};
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-              rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 1));
-              rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 2));
-              const float m_new = fmaxf(m[t][h], rmax[h]);  // finite: a live warp sees at least one of its keys
-              corr[h] = __expf(m[t][h] - m_new);
-              m[t][h] = m_new;
+            for (int e = 0; e < 4; ++e) {
+              const int key = kt0 + key0 + j * 8 + (lane & 3) * 2 + (e & 1);
+              s[j][e] = key <= pos && (key >= lo || key < p.keep) ? s[j][e] * p.scale : -INFINITY;
             }
+          float rmax[2] = {fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1])),
+                           fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]))};
+          float corr[2], rsum[2] = {0.f, 0.f};
 #pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                s[t][j][e] = __expf(s[t][j][e] - m[t][e >> 1]);
-                rsum[e >> 1] += s[t][j][e];
-              }
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-              rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 1);
-              rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 2);
-              l[t][h] = l[t][h] * corr[h] + rsum[h];
-            }
-#pragma unroll
-            for (int i = 0; i < HD / 8; ++i) {
-              acc[t][i][0] *= corr[0]; acc[t][i][1] *= corr[0];
-              acc[t][i][2] *= corr[1]; acc[t][i][3] *= corr[1];
-            }
-            pf[t][0] = pack_bf16(s[t][0][0], s[t][0][1]); pf[t][1] = pack_bf16(s[t][0][2], s[t][0][3]);
-            pf[t][2] = pack_bf16(s[t][1][0], s[t][1][1]); pf[t][3] = pack_bf16(s[t][1][2], s[t][1][3]);
+          for (int h = 0; h < 2; ++h) {
+            rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 1));
+            rmax[h] = fmaxf(rmax[h], __shfl_xor_sync(0xffffffffu, rmax[h], 2));
+            const float m_new = fmaxf(m[h], rmax[h]);  // finite: a live warp sees at least one of its keys
+            corr[h] = __expf(m[h] - m_new);
+            m[h] = m_new;
           }
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              s[j][e] = __expf(s[j][e] - m[e >> 1]);
+              rsum[e >> 1] += s[j][e];
+            }
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 1);
+            rsum[h] += __shfl_xor_sync(0xffffffffu, rsum[h], 2);
+            l[h] = l[h] * corr[h] + rsum[h];
+          }
+#pragma unroll
+          for (int i = 0; i < HD / 8; ++i) {
+            acc[i][0] *= corr[0]; acc[i][1] *= corr[0];
+            acc[i][2] *= corr[1]; acc[i][3] *= corr[1];
+          }
+          pf[0] = pack_bf16(s[0][0], s[0][1]); pf[1] = pack_bf16(s[0][2], s[0][3]);
+          pf[2] = pack_bf16(s[1][0], s[1][1]); pf[3] = pack_bf16(s[1][2], s[1][3]);
         }
       } else {
         const int c = c_lo + item - p.KV;  // rows of other value heads weigh nothing here
-        const int first_row = c * p.G - head0;
-#pragma unroll
-        for (int t = 0; t < MT; ++t) {
-          if (first_row >= (t + 1) * 16 || first_row + p.G <= t * 16) continue;  // none of this tile's rows
-          const uint32_t own[4] = {owner[t][0] == c ? pf[t][0] : 0u, owner[t][1] == c ? pf[t][1] : 0u,
-                                   owner[t][0] == c ? pf[t][2] : 0u, owner[t][1] == c ? pf[t][3] : 0u};
-          pv_16keys<HD>(acc[t], own, stage(n), key0, lane);
-        }
+        const uint32_t own[4] = {owner[0] == c ? pf[0] : 0u, owner[1] == c ? pf[1] : 0u, owner[0] == c ? pf[2] : 0u,
+                                 owner[1] == c ? pf[3] : 0u};
+        const int first_row = c * p.G - head0 - group * 16;
+        if (first_row < 16 && first_row + p.G > 0) pv_16keys<HD>(acc, own, stage(n), key0, lane);  // (else none of this group's rows)
       }
     }
     if (++item == items) { item = 0; ++tile; }
@@ -286,23 +269,21 @@ parts_decode_kernel(const PartsParams p) {
   {
     const int g = lane >> 2, q = lane & 3;
 #pragma unroll
-    for (int t = 0; t < MT; ++t)
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int rr = t * 16 + h * 8 + g, at = warp * kRows + rr;
-        if (q == 0) {
-          mm[at] = m[t][h];
-          ml[at] = l[t][h];
-        }
-        if (rr < gc) {
-#pragma unroll
-          for (int i = 0; i < HD / 8; ++i)
-            *reinterpret_cast<float2*>(ma + (size_t)at * HD + i * 8 + q * 2) = make_float2(acc[t][i][2 * h], acc[t][i][2 * h + 1]);
-        }
+    for (int h = 0; h < 2; ++h) {
+      const int rr = group * 16 + h * 8 + g, at = (warp & 3) * kRows + rr;
+      if (q == 0) {
+        mm[at] = m[h];
+        ml[at] = l[h];
       }
+      if (rr < gc) {
+#pragma unroll
+        for (int i = 0; i < HD / 8; ++i)
+          *reinterpret_cast<float2*>(ma + (size_t)at * HD + i * 8 + q * 2) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
+      }
+    }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < gc * HD; i += kDecodeThreads) {
+  for (int i = threadIdx.x; i < gc * HD; i += kThreads) {
     const int qr = i / HD, col = i - qr * HD;
     float mx = -INFINITY;
 #pragma unroll
@@ -521,9 +502,9 @@ parts_prefill_kernel(const PartsParams p) {
 
 constexpr size_t kMaxSmem = 227 * 1024;
 
-int decode_tiles(int H) { return H > 16 ? 2 : 1; }
+int decode_groups(int H) { return H > 16 ? 2 : 1; }
 size_t decode_smem(int hd, int H, int KV, int stages) {
-  return (size_t)stages * kKeyTile * hd * 2 + (size_t)KV * decode_tiles(H) * 16 * hd * 2;
+  return (size_t)stages * kKeyTile * hd * 2 + (size_t)KV * decode_groups(H) * 16 * hd * 2;
 }
 // four stages where two blocks then share an SM, else eight where they fit (one block keeps the copies going)
 int decode_stages(int hd, int H, int KV) {
@@ -531,7 +512,7 @@ int decode_stages(int hd, int H, int KV) {
 }
 // heads per block: whole groups where they fit its rows, so that no value head is read twice
 int decode_heads(int H, int KV) {
-  const int G = H / KV, most = 16 * decode_tiles(H);
+  const int G = H / KV, most = 16 * decode_groups(H);
   return H <= most ? H : (G <= most ? most / G * G : most);
 }
 size_t prefill_smem(int hd, int KV, bool stream) {
@@ -549,7 +530,7 @@ int start(Kernel kern, dim3 grid, int threads, size_t smem, cudaStream_t stream,
 
 template <typename F>
 auto with_decode_kernel(int hd, int H, int KV, F&& use) {
-  const bool two = decode_tiles(H) == 2, eight = decode_stages(hd, H, KV) == 8;
+  const bool two = decode_groups(H) == 2, eight = decode_stages(hd, H, KV) == 8;
 #define ASB_PICK(HD) \
   (two ? (eight ? use(parts_decode_kernel<HD, 2, 8>) : use(parts_decode_kernel<HD, 2, 4>)) \
        : (eight ? use(parts_decode_kernel<HD, 1, 8>) : use(parts_decode_kernel<HD, 1, 4>)))
@@ -565,7 +546,7 @@ int launch_parts(PartsParams p, int run_decode, int run_prefill, cudaStream_t st
     if (p.HC > 65535) return asb::fail("attention_parts: too many heads");
     dim3 grid(p.short_rows > 0 ? p.short_rows : p.T, p.HC, p.NP);
     const size_t smem = decode_smem(HD, p.H, p.KV, decode_stages(HD, p.H, p.KV));
-    if (int rc = with_decode_kernel(HD, p.H, p.KV, [&](auto kern) { return start(kern, grid, kDecodeThreads, smem, stream, p, "parts_decode"); })) return rc;
+    if (int rc = with_decode_kernel(HD, p.H, p.KV, [&](auto kern) { return start(kern, grid, 128 * decode_groups(p.H), smem, stream, p, "parts_decode"); })) return rc;
   }
   if (run_prefill) {
     p.GC = p.G < 16 ? p.G : 16;
@@ -599,7 +580,7 @@ extern "C" int asb_attention_parts_resident(int hd, int H, int KV) {
   const size_t smem = decode_smem(hd, H, KV, decode_stages(hd, H, KV));
   const cudaError_t e = with_decode_kernel(hd, H, KV, [&](auto kern) {
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kern, kDecodeThreads, smem);
+    return cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kern, 128 * decode_groups(H), smem);
   });
   return e == cudaSuccess ? per_sm * sms : 0;
 }

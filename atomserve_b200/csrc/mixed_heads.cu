@@ -222,11 +222,12 @@ mixed_heads_prepare_kernel(const MixedParams p) {
 // The usual form: neighbouring pairs (or no rotation), head sizes that are multiples of 8. A thread keeps
 // its vectors of four columns in registers from the projection to where they belong: both entries of a
 // pair lie in one vector, so norm and rotation touch no shared memory; keys and values go to their
-// pages and queries to shared memory for the mix. kPer: vectors a thread. R and E: the group's heads
+// pages and queries to shared memory for the mix. A block takes several tokens, one after another, and
+// holds the biases, gains and mixing weights for all of them. kPer: vectors a thread. R and E: the group's heads
 // whose E entries a thread holds while it walks the output heads.
 template <typename T, int R, int E, int kPer>
-__global__ void __launch_bounds__(256, kPer <= 4 ? 3 : 2)
-mixed_heads_prepare_vec_kernel(const MixedParams p) {
+__global__ void __launch_bounds__(256, kPer <= 6 ? 3 : 2)
+mixed_heads_prepare_vec_kernel(const MixedParams p, int tokens) {
   extern __shared__ __align__(16) float smem[];
   __shared__ float scratch[2][8];
   const int H = p.H, KV = p.KV, hd = p.hd, dim = p.dim;
@@ -248,133 +249,146 @@ mixed_heads_prepare_vec_kernel(const MixedParams p) {
   }
   asb::pdl_wait();
   asb::pdl_launch_dependents();
-  const int t = blockIdx.x, half = p.rotary_dim >> 1;
-  float v[kPer][4];
-  float sq = 0.f, sk = 0.f;
+  const int half = p.rotary_dim >> 1;
+  // (a token's scratch and angles are written when everybody is past the barrier behind the last reads of
+  // the token before, its queries when everybody is past that token's mix: the first barrier below)
+  for (int t = blockIdx.x; t < tokens; t += gridDim.x) {
+    float v[kPer][4];
+    float sq = 0.f, sk = 0.f;
 #pragma unroll
-  for (int u = 0; u < kPer; ++u) {
-    const int i = threadIdx.x + u * 256;
-    if (i < total) column<T, 4>(p, t, 4 * i, v[u], false);
-  }
-  const float position = (float)__ldcg(p.positions + t);
-  for (int i = threadIdx.x; i < half; i += 256) sincosf(position * p.inv_freq[i], &cs[half + i], &cs[i]);
-  const int slot = p.slots ? __ldcg(p.slots + t) : -1;
-  const bool store = p.k_cache && slot >= 0;
-#pragma unroll
-  for (int u = 0; u < kPer; ++u) {
-    const int i = threadIdx.x + u * 256;
-    if (i >= total) continue;
-    v[u][0] += bias[u].x; v[u][1] += bias[u].y; v[u][2] += bias[u].z; v[u][3] += bias[u].w;
-    const float ss = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
-    if (i < nq) sq += ss;
-    else if (i < nq + nk) sk += ss;
-  }
-  sq = asb::warp_sum(sq);
-  sk = asb::warp_sum(sk);
-  if ((threadIdx.x & 31) == 0) {
-    scratch[0][threadIdx.x >> 5] = sq;
-    scratch[1][threadIdx.x >> 5] = sk;
-  }
-  __syncthreads();  // (the angles too)
-  float inv_q = 1.f, inv_k = 1.f;
-  if (p.q_gain) {
-    sq = sk = 0.f;
-#pragma unroll
-    for (int w = 0; w < 8; ++w) {
-      sq += scratch[0][w];
-      sk += scratch[1][w];
+    for (int u = 0; u < kPer; ++u) {
+      const int i = threadIdx.x + u * 256;
+      if (i < total) column<T, 4>(p, t, 4 * i, v[u], false);
     }
-    inv_q = 1.f / sqrtf(sq / (float)(H * dim) + p.eps);
-    inv_k = 1.f / sqrtf(sk / (float)(KV * dim) + p.eps);
-  }
-  const size_t page = store ? slot / p.bs : 0, off = store ? slot % p.bs : 0;
+    const float position = (float)__ldcg(p.positions + t);
+    for (int i = threadIdx.x; i < half; i += 256) sincosf(position * p.inv_freq[i], &cs[half + i], &cs[i]);
+    const int slot = p.slots ? __ldcg(p.slots + t) : -1;
+    const bool store = p.k_cache && slot >= 0;
 #pragma unroll
-  for (int u = 0; u < kPer; ++u) {
-    const int i = threadIdx.x + u * 256;
-    if (i >= total) continue;
-    if (i < nq + nk) {
-      const bool query = i < nq;
-      const int col = 4 * (query ? i : i - nq), h = col / dim, e = col - h * dim;
-      const float inv = query ? inv_q : inv_k;
-      const float g[4] = {gain[u].x, gain[u].y, gain[u].z, gain[u].w};
-      float w[4];
+    for (int u = 0; u < kPer; ++u) {
+      const int i = threadIdx.x + u * 256;
+      if (i >= total) continue;
+      v[u][0] += bias[u].x; v[u][1] += bias[u].y; v[u][2] += bias[u].z; v[u][3] += bias[u].w;
+      const float ss = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
+      if (i < nq) sq += ss;
+      else if (i < nq + nk) sk += ss;
+    }
+    sq = asb::warp_sum(sq);
+    sk = asb::warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) {
+      scratch[0][threadIdx.x >> 5] = sq;
+      scratch[1][threadIdx.x >> 5] = sk;
+    }
+    __syncthreads();  // (the angles too)
+    float inv_q = 1.f, inv_k = 1.f;
+    if (p.q_gain) {
+      sq = sk = 0.f;
 #pragma unroll
-      for (int k = 0; k < 4; ++k) w[k] = v[u][k] * inv * g[k];
+      for (int w = 0; w < 8; ++w) {
+        sq += scratch[0][w];
+        sk += scratch[1][w];
+      }
+      inv_q = 1.f / sqrtf(sq / (float)(H * dim) + p.eps);
+      inv_k = 1.f / sqrtf(sk / (float)(KV * dim) + p.eps);
+    }
+    const size_t page = store ? slot / p.bs : 0, off = store ? slot % p.bs : 0;
 #pragma unroll
-      for (int k = 0; k < 4; k += 2) {
-        const int pair = (e + k) >> 1;
-        if (pair < half) {
-          const float c = cs[pair], s = cs[half + pair], a = w[k], b = w[k + 1];
-          w[k] = a * c - b * s;
-          w[k + 1] = b * c + a * s;
+    for (int u = 0; u < kPer; ++u) {
+      const int i = threadIdx.x + u * 256;
+      if (i >= total) continue;
+      if (i < nq + nk) {
+        const bool query = i < nq;
+        const int col = 4 * (query ? i : i - nq), h = col / dim, e = col - h * dim;
+        const float inv = query ? inv_q : inv_k;
+        const float g[4] = {gain[u].x, gain[u].y, gain[u].z, gain[u].w};
+        float w[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) w[k] = v[u][k] * inv * g[k];
+#pragma unroll
+        for (int k = 0; k < 4; k += 2) {
+          const int pair = (e + k) >> 1;
+          if (pair < half) {
+            const float c = cs[pair], s = cs[half + pair], a = w[k], b = w[k + 1];
+            w[k] = a * c - b * s;
+            w[k + 1] = b * c + a * s;
+          }
         }
-      }
-      if (query) *reinterpret_cast<float4*>(q_s + h * hd + e) = make_float4(w[0], w[1], w[2], w[3]);
-      else if (store) store4<T>((T*)p.k_cache + ((page * KV + h) * p.bs + off) * hd + e, w);
-    } else {
-      const int col = 4 * (i - nq - nk), h = col / p.vdim, e = col - h * p.vdim;
-      const size_t at = (size_t)t * KV * p.vdim + col;
-      if (p.v_out) store4<T>((T*)p.v_out + at, v[u]);
-      if (p.v_first) {
-        float f[4];
-        load4<T>((const T*)p.v_first + at, f);
+        if (query) *reinterpret_cast<float4*>(q_s + h * hd + e) = make_float4(w[0], w[1], w[2], w[3]);
+        else if (store) store4<T>((T*)p.k_cache + ((page * KV + h) * p.bs + off) * hd + e, w);
+      } else {
+        const int col = 4 * (i - nq - nk), h = col / p.vdim, e = col - h * p.vdim;
+        const size_t at = (size_t)t * KV * p.vdim + col;
+        if (p.v_out) store4<T>((T*)p.v_out + at, v[u]);
+        if (p.v_first) {
+          float f[4];
+          load4<T>((const T*)p.v_first + at, f);
 #pragma unroll
-        for (int k = 0; k < 4; ++k) v[u][k] = (1.f - p.lambda) * v[u][k] + p.lambda * f[k];
+          for (int k = 0; k < 4; ++k) v[u][k] = (1.f - p.lambda) * v[u][k] + p.lambda * f[k];
+        }
+        if (store) store4<T>((T*)p.v_cache + ((page * KV + h) * p.bs + off) * hd + e, v[u]);
       }
-      if (store) store4<T>((T*)p.v_cache + ((page * KV + h) * p.bs + off) * hd + e, v[u]);
     }
-  }
-  if (store) {  // zeros behind what a head holds
-    const float zero[4] = {0.f, 0.f, 0.f, 0.f};
-    const int kz = (hd - dim) >> 2, vz = (hd - p.vdim) >> 2;
-    for (int i = threadIdx.x; i < KV * kz; i += 256) store4<T>((T*)p.k_cache + ((page * KV + i / kz) * p.bs + off) * hd + dim + i % kz * 4, zero);
-    for (int i = threadIdx.x; i < KV * vz; i += 256) store4<T>((T*)p.v_cache + ((page * KV + i / vz) * p.bs + off) * hd + p.vdim + i % vz * 4, zero);
-  }
-  __syncthreads();
-  T* q_out = (T*)p.q_out + (size_t)t * H * KV * hd;
-  // (part, E entries) per thread; the threads that are left over share the output heads
-  const int per = hd / E, items = KV * per, lanes = items < 256 ? 256 / items : 1;
-  if ((int)threadIdx.x >= items * lanes) return;
-  for (int item = threadIdx.x % items; item < items; item += 256) {
-    const int c = item / per, e = (item - c * per) * E;
-    float q[R][E];
-#pragma unroll
-    for (int g = 0; g < R; ++g)
-#pragma unroll
-      for (int k = 0; k < E; k += 4) {
-        const float4 f = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e + k);
-        q[g][k] = f.x; q[g][k + 1] = f.y; q[g][k + 2] = f.z; q[g][k + 3] = f.w;
-      }
-    for (int h = items < 256 ? threadIdx.x / items : 0; h < H; h += lanes) {
-      float sum[E], w[R];
-#pragma unroll
-      for (int g = 0; g < R; ++g) w[g] = talk_s[h * H + c * R + g];
-#pragma unroll
-      for (int k = 0; k < E; ++k) sum[k] = 0.f;
+    if (store) {  // zeros behind what a head holds
+      const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+      const int kz = (hd - dim) >> 2, vz = (hd - p.vdim) >> 2;
+      for (int i = threadIdx.x; i < KV * kz; i += 256) store4<T>((T*)p.k_cache + ((page * KV + i / kz) * p.bs + off) * hd + dim + i % kz * 4, zero);
+      for (int i = threadIdx.x; i < KV * vz; i += 256) store4<T>((T*)p.v_cache + ((page * KV + i / vz) * p.bs + off) * hd + p.vdim + i % vz * 4, zero);
+    }
+    __syncthreads();
+    T* q_out = (T*)p.q_out + (size_t)t * H * KV * hd;
+    // (part, E entries) per thread; the threads that are left over share the output heads
+    const int per = hd / E, items = KV * per, lanes = items < 256 ? 256 / items : 1;
+    for (int item = (int)threadIdx.x < items * lanes ? threadIdx.x % items : items; item < items; item += 256) {
+      const int c = item / per, e = (item - c * per) * E;
+      float q[R][E];
 #pragma unroll
       for (int g = 0; g < R; ++g)
 #pragma unroll
-        for (int k = 0; k < E; ++k) sum[k] = fmaf(w[g], q[g][k], sum[k]);
-      T* at = q_out + ((size_t)h * KV + c) * hd + e;
-      if constexpr (E == 8) store8<T>(at, sum);
-      else store4<T>(at, sum);
+        for (int k = 0; k < E; k += 4) {
+          const float4 f = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e + k);
+          q[g][k] = f.x; q[g][k + 1] = f.y; q[g][k + 2] = f.z; q[g][k + 3] = f.w;
+        }
+      for (int h = items < 256 ? threadIdx.x / items : 0; h < H; h += lanes) {
+        float sum[E], w[R];
+#pragma unroll
+        for (int g = 0; g < R; g += R >= 4 ? 4 : 1) {
+          const float* at = talk_s + h * H + c * R + g;
+          if constexpr (R >= 4) {
+            const float4 f = *reinterpret_cast<const float4*>(at);
+            w[g] = f.x; w[g + 1] = f.y; w[g + 2] = f.z; w[g + 3] = f.w;
+          } else {
+            w[g] = *at;
+          }
+        }
+#pragma unroll
+        for (int k = 0; k < E; ++k) sum[k] = 0.f;
+#pragma unroll
+        for (int g = 0; g < R; ++g)
+#pragma unroll
+          for (int k = 0; k < E; ++k) sum[k] = fmaf(w[g], q[g][k], sum[k]);
+        T* at = q_out + ((size_t)h * KV + c) * hd + e;
+        if constexpr (E == 8) store8<T>(at, sum);
+        else store4<T>(at, sum);
+      }
     }
   }
 }
 
-template <typename T, typename Kernel>
-int start(Kernel kern, const MixedParams& p, int tokens, size_t smem, cudaStream_t stream) {
+template <typename Kernel, typename... More>
+int start(Kernel kern, const MixedParams& p, int blocks, size_t smem, cudaStream_t stream, More... more) {
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return asb::fail("mixed_heads_prepare: shared memory %zu: %s", smem, cudaGetErrorString(e));
-  asb::launch(kern, tokens, 256, smem, stream, p);
+  asb::launch(kern, blocks, 256, smem, stream, p, more...);
   return asb::check_launch("mixed_heads_prepare");
 }
 
 template <typename T, int R, int E>
 int start_vec(const MixedParams& p, int tokens, int vectors, size_t smem, cudaStream_t stream) {
-  if (vectors <= 2 * 256) return start<T>(mixed_heads_prepare_vec_kernel<T, R, E, 2>, p, tokens, smem, stream);
-  if (vectors <= 4 * 256) return start<T>(mixed_heads_prepare_vec_kernel<T, R, E, 4>, p, tokens, smem, stream);
-  return start<T>(mixed_heads_prepare_vec_kernel<T, R, E, 8>, p, tokens, smem, stream);
+  const int most = 148 * (vectors <= 6 * 256 ? 3 : 2), blocks = tokens < most ? tokens : most;  // one wave
+  if (vectors <= 2 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 2>, p, blocks, smem, stream, tokens);
+  if (vectors <= 4 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 4>, p, blocks, smem, stream, tokens);
+  if (vectors <= 6 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 6>, p, blocks, smem, stream, tokens);
+  return start(mixed_heads_prepare_vec_kernel<T, R, E, 8>, p, blocks, smem, stream, tokens);
 }
 
 template <typename T>
@@ -391,8 +405,8 @@ int dispatch(const MixedParams& p, int tokens, cudaStream_t stream) {
   if (eight && G == 2) return start_vec<T, 2, 8>(p, tokens, vectors, smem, stream);
   if (eight && G == 4) return start_vec<T, 4, 8>(p, tokens, vectors, smem, stream);
   if (eight && G == 8) return start_vec<T, 8, 4>(p, tokens, vectors, smem, stream);
-  if (four) return start<T>(mixed_heads_prepare_kernel<T, 4>, p, tokens, smem, stream);
-  return start<T>(mixed_heads_prepare_kernel<T, 1>, p, tokens, smem, stream);
+  if (four) return start(mixed_heads_prepare_kernel<T, 4>, p, tokens, smem, stream);
+  return start(mixed_heads_prepare_kernel<T, 1>, p, tokens, smem, stream);
 }
 
 }  // namespace
