@@ -222,12 +222,11 @@ mixed_heads_prepare_kernel(const MixedParams p) {
 // The usual form: neighbouring pairs (or no rotation), head sizes that are multiples of 8. A thread keeps
 // its vectors of four columns in registers from the projection to where they belong: both entries of a
 // pair lie in one vector, so norm and rotation touch no shared memory; keys and values go to their
-// pages and queries to shared memory for the mix. A block takes several tokens, one after another, and
-// holds the biases, gains and mixing weights for all of them. kPer: vectors a thread. R and E: the group's heads
+// pages and queries to shared memory for the mix. kPer: vectors a thread. R and E: the group's heads
 // whose E entries a thread holds while it walks the output heads.
 template <typename T, int R, int E, int kPer>
 __global__ void __launch_bounds__(256, kPer <= 6 ? 3 : 2)
-mixed_heads_prepare_vec_kernel(const MixedParams p, int tokens) {
+mixed_heads_prepare_vec_kernel(const MixedParams p) {
   extern __shared__ __align__(16) float smem[];
   __shared__ float scratch[2][8];
   const int H = p.H, KV = p.KV, hd = p.hd, dim = p.dim;
@@ -238,157 +237,147 @@ mixed_heads_prepare_vec_kernel(const MixedParams p, int tokens) {
   // what no kernel writes is read before the wait
   for (int i = threadIdx.x; i < H * H; i += 256) talk_s[i] = p.talk[i];
   for (int i = threadIdx.x; i < H * (hd - dim); i += 256) q_s[i / (hd - dim) * hd + dim + i % (hd - dim)] = 0.f;
-  float4 bias[kPer], gain[kPer];
-#pragma unroll
-  for (int u = 0; u < kPer; ++u) {
-    const int i = threadIdx.x + u * 256;
-    bias[u] = p.bias && i < total ? *reinterpret_cast<const float4*>(p.bias + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
-    gain[u] = make_float4(1.f, 1.f, 1.f, 1.f);
-    if (p.q_gain && i < nq) gain[u] = *reinterpret_cast<const float4*>(p.q_gain + 4 * i);
-    else if (p.q_gain && i < nq + nk) gain[u] = *reinterpret_cast<const float4*>(p.k_gain + 4 * (i - nq));
-  }
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   const int half = p.rotary_dim >> 1;
-  // (a token's scratch and angles are written when everybody is past the barrier behind the last reads of
-  // the token before, its queries when everybody is past that token's mix: the first barrier below)
-  for (int t = blockIdx.x; t < tokens; t += gridDim.x) {
-    float v[kPer][4];
-    float sq = 0.f, sk = 0.f;
+  const int t = blockIdx.x;
+  float v[kPer][4];
+  float sq = 0.f, sk = 0.f;
 #pragma unroll
-    for (int u = 0; u < kPer; ++u) {
-      const int i = threadIdx.x + u * 256;
-      if (i < total) column<T, 4>(p, t, 4 * i, v[u], false);
-    }
-    const float position = (float)__ldcg(p.positions + t);
-    for (int i = threadIdx.x; i < half; i += 256) sincosf(position * p.inv_freq[i], &cs[half + i], &cs[i]);
-    const int slot = p.slots ? __ldcg(p.slots + t) : -1;
-    const bool store = p.k_cache && slot >= 0;
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    if (i < total) column<T, 4>(p, t, 4 * i, v[u], false);
+  }
+  const float position = (float)__ldcg(p.positions + t);
+  for (int i = threadIdx.x; i < half; i += 256) sincosf(position * p.inv_freq[i], &cs[half + i], &cs[i]);
+  const int slot = p.slots ? __ldcg(p.slots + t) : -1;
+  const bool store = p.k_cache && slot >= 0;
 #pragma unroll
-    for (int u = 0; u < kPer; ++u) {
-      const int i = threadIdx.x + u * 256;
-      if (i >= total) continue;
-      v[u][0] += bias[u].x; v[u][1] += bias[u].y; v[u][2] += bias[u].z; v[u][3] += bias[u].w;
-      const float ss = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
-      if (i < nq) sq += ss;
-      else if (i < nq + nk) sk += ss;
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    if (i >= total) continue;
+    if (p.bias) {
+      const float4 b = *reinterpret_cast<const float4*>(p.bias + 4 * i);
+      v[u][0] += b.x; v[u][1] += b.y; v[u][2] += b.z; v[u][3] += b.w;
     }
-    sq = asb::warp_sum(sq);
-    sk = asb::warp_sum(sk);
-    if ((threadIdx.x & 31) == 0) {
-      scratch[0][threadIdx.x >> 5] = sq;
-      scratch[1][threadIdx.x >> 5] = sk;
-    }
-    __syncthreads();  // (the angles too)
-    float inv_q = 1.f, inv_k = 1.f;
-    if (p.q_gain) {
-      sq = sk = 0.f;
+    const float ss = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
+    if (i < nq) sq += ss;
+    else if (i < nq + nk) sk += ss;
+  }
+  sq = asb::warp_sum(sq);
+  sk = asb::warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    scratch[0][threadIdx.x >> 5] = sq;
+    scratch[1][threadIdx.x >> 5] = sk;
+  }
+  __syncthreads();  // (the angles too)
+  float inv_q = 1.f, inv_k = 1.f;
+  if (p.q_gain) {
+    sq = sk = 0.f;
 #pragma unroll
-      for (int w = 0; w < 8; ++w) {
-        sq += scratch[0][w];
-        sk += scratch[1][w];
-      }
-      inv_q = 1.f / sqrtf(sq / (float)(H * dim) + p.eps);
-      inv_k = 1.f / sqrtf(sk / (float)(KV * dim) + p.eps);
+    for (int w = 0; w < 8; ++w) {
+      sq += scratch[0][w];
+      sk += scratch[1][w];
     }
-    const size_t page = store ? slot / p.bs : 0, off = store ? slot % p.bs : 0;
+    inv_q = 1.f / sqrtf(sq / (float)(H * dim) + p.eps);
+    inv_k = 1.f / sqrtf(sk / (float)(KV * dim) + p.eps);
+  }
+  const size_t page = store ? slot / p.bs : 0, off = store ? slot % p.bs : 0;
 #pragma unroll
-    for (int u = 0; u < kPer; ++u) {
-      const int i = threadIdx.x + u * 256;
-      if (i >= total) continue;
-      if (i < nq + nk) {
-        const bool query = i < nq;
-        const int col = 4 * (query ? i : i - nq), h = col / dim, e = col - h * dim;
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * 256;
+    if (i >= total) continue;
+    if (i < nq + nk) {
+      const bool query = i < nq;
+      const int col = 4 * (query ? i : i - nq), h = col / dim, e = col - h * dim;
+      float w[4] = {v[u][0], v[u][1], v[u][2], v[u][3]};
+      if (p.q_gain) {
+        const float4 g = *reinterpret_cast<const float4*>((query ? p.q_gain : p.k_gain) + col);
         const float inv = query ? inv_q : inv_k;
-        const float g[4] = {gain[u].x, gain[u].y, gain[u].z, gain[u].w};
-        float w[4];
-#pragma unroll
-        for (int k = 0; k < 4; ++k) w[k] = v[u][k] * inv * g[k];
-#pragma unroll
-        for (int k = 0; k < 4; k += 2) {
-          const int pair = (e + k) >> 1;
-          if (pair < half) {
-            const float c = cs[pair], s = cs[half + pair], a = w[k], b = w[k + 1];
-            w[k] = a * c - b * s;
-            w[k + 1] = b * c + a * s;
-          }
-        }
-        if (query) *reinterpret_cast<float4*>(q_s + h * hd + e) = make_float4(w[0], w[1], w[2], w[3]);
-        else if (store) store4<T>((T*)p.k_cache + ((page * KV + h) * p.bs + off) * hd + e, w);
-      } else {
-        const int col = 4 * (i - nq - nk), h = col / p.vdim, e = col - h * p.vdim;
-        const size_t at = (size_t)t * KV * p.vdim + col;
-        if (p.v_out) store4<T>((T*)p.v_out + at, v[u]);
-        if (p.v_first) {
-          float f[4];
-          load4<T>((const T*)p.v_first + at, f);
-#pragma unroll
-          for (int k = 0; k < 4; ++k) v[u][k] = (1.f - p.lambda) * v[u][k] + p.lambda * f[k];
-        }
-        if (store) store4<T>((T*)p.v_cache + ((page * KV + h) * p.bs + off) * hd + e, v[u]);
+        w[0] *= inv * g.x; w[1] *= inv * g.y; w[2] *= inv * g.z; w[3] *= inv * g.w;
       }
+#pragma unroll
+      for (int k = 0; k < 4; k += 2) {
+        const int pair = (e + k) >> 1;
+        if (pair < half) {
+          const float c = cs[pair], s = cs[half + pair], a = w[k], b = w[k + 1];
+          w[k] = a * c - b * s;
+          w[k + 1] = b * c + a * s;
+        }
+      }
+      if (query) *reinterpret_cast<float4*>(q_s + h * hd + e) = make_float4(w[0], w[1], w[2], w[3]);
+      else if (store) store4<T>((T*)p.k_cache + ((page * KV + h) * p.bs + off) * hd + e, w);
+    } else {
+      const int col = 4 * (i - nq - nk), h = col / p.vdim, e = col - h * p.vdim;
+      const size_t at = (size_t)t * KV * p.vdim + col;
+      if (p.v_out) store4<T>((T*)p.v_out + at, v[u]);
+      if (p.v_first) {
+        float f[4];
+        load4<T>((const T*)p.v_first + at, f);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[u][k] = (1.f - p.lambda) * v[u][k] + p.lambda * f[k];
+      }
+      if (store) store4<T>((T*)p.v_cache + ((page * KV + h) * p.bs + off) * hd + e, v[u]);
     }
-    if (store) {  // zeros behind what a head holds
-      const float zero[4] = {0.f, 0.f, 0.f, 0.f};
-      const int kz = (hd - dim) >> 2, vz = (hd - p.vdim) >> 2;
-      for (int i = threadIdx.x; i < KV * kz; i += 256) store4<T>((T*)p.k_cache + ((page * KV + i / kz) * p.bs + off) * hd + dim + i % kz * 4, zero);
-      for (int i = threadIdx.x; i < KV * vz; i += 256) store4<T>((T*)p.v_cache + ((page * KV + i / vz) * p.bs + off) * hd + p.vdim + i % vz * 4, zero);
-    }
-    __syncthreads();
-    T* q_out = (T*)p.q_out + (size_t)t * H * KV * hd;
-    // (part, E entries) per thread; the threads that are left over share the output heads
-    const int per = hd / E, items = KV * per, lanes = items < 256 ? 256 / items : 1;
-    for (int item = (int)threadIdx.x < items * lanes ? threadIdx.x % items : items; item < items; item += 256) {
-      const int c = item / per, e = (item - c * per) * E;
-      float q[R][E];
+  }
+  if (store) {  // zeros behind what a head holds
+    const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+    const int kz = (hd - dim) >> 2, vz = (hd - p.vdim) >> 2;
+    for (int i = threadIdx.x; i < KV * kz; i += 256) store4<T>((T*)p.k_cache + ((page * KV + i / kz) * p.bs + off) * hd + dim + i % kz * 4, zero);
+    for (int i = threadIdx.x; i < KV * vz; i += 256) store4<T>((T*)p.v_cache + ((page * KV + i / vz) * p.bs + off) * hd + p.vdim + i % vz * 4, zero);
+  }
+  __syncthreads();
+  T* q_out = (T*)p.q_out + (size_t)t * H * KV * hd;
+  // (part, E entries) per thread; the threads that are left over share the output heads
+  const int per = hd / E, items = KV * per, lanes = items < 256 ? 256 / items : 1;
+  for (int item = (int)threadIdx.x < items * lanes ? threadIdx.x % items : items; item < items; item += 256) {
+    const int c = item / per, e = (item - c * per) * E;
+    float q[R][E];
+#pragma unroll
+    for (int g = 0; g < R; ++g)
+#pragma unroll
+      for (int k = 0; k < E; k += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e + k);
+        q[g][k] = f.x; q[g][k + 1] = f.y; q[g][k + 2] = f.z; q[g][k + 3] = f.w;
+      }
+    for (int h = items < 256 ? threadIdx.x / items : 0; h < H; h += lanes) {
+      float sum[E], w[R];
+#pragma unroll
+      for (int g = 0; g < R; g += R >= 4 ? 4 : 1) {
+        const float* at = talk_s + h * H + c * R + g;
+        if constexpr (R >= 4) {
+          const float4 f = *reinterpret_cast<const float4*>(at);
+          w[g] = f.x; w[g + 1] = f.y; w[g + 2] = f.z; w[g + 3] = f.w;
+        } else {
+          w[g] = *at;
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < E; ++k) sum[k] = 0.f;
 #pragma unroll
       for (int g = 0; g < R; ++g)
 #pragma unroll
-        for (int k = 0; k < E; k += 4) {
-          const float4 f = *reinterpret_cast<const float4*>(q_s + (c * R + g) * hd + e + k);
-          q[g][k] = f.x; q[g][k + 1] = f.y; q[g][k + 2] = f.z; q[g][k + 3] = f.w;
-        }
-      for (int h = items < 256 ? threadIdx.x / items : 0; h < H; h += lanes) {
-        float sum[E], w[R];
-#pragma unroll
-        for (int g = 0; g < R; g += R >= 4 ? 4 : 1) {
-          const float* at = talk_s + h * H + c * R + g;
-          if constexpr (R >= 4) {
-            const float4 f = *reinterpret_cast<const float4*>(at);
-            w[g] = f.x; w[g + 1] = f.y; w[g + 2] = f.z; w[g + 3] = f.w;
-          } else {
-            w[g] = *at;
-          }
-        }
-#pragma unroll
-        for (int k = 0; k < E; ++k) sum[k] = 0.f;
-#pragma unroll
-        for (int g = 0; g < R; ++g)
-#pragma unroll
-          for (int k = 0; k < E; ++k) sum[k] = fmaf(w[g], q[g][k], sum[k]);
-        T* at = q_out + ((size_t)h * KV + c) * hd + e;
-        if constexpr (E == 8) store8<T>(at, sum);
-        else store4<T>(at, sum);
-      }
+        for (int k = 0; k < E; ++k) sum[k] = fmaf(w[g], q[g][k], sum[k]);
+      T* at = q_out + ((size_t)h * KV + c) * hd + e;
+      if constexpr (E == 8) store8<T>(at, sum);
+      else store4<T>(at, sum);
     }
   }
 }
 
-template <typename Kernel, typename... More>
-int start(Kernel kern, const MixedParams& p, int blocks, size_t smem, cudaStream_t stream, More... more) {
+template <typename Kernel>
+int start(Kernel kern, const MixedParams& p, int tokens, size_t smem, cudaStream_t stream) {
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return asb::fail("mixed_heads_prepare: shared memory %zu: %s", smem, cudaGetErrorString(e));
-  asb::launch(kern, blocks, 256, smem, stream, p, more...);
+  asb::launch(kern, tokens, 256, smem, stream, p);
   return asb::check_launch("mixed_heads_prepare");
 }
 
 template <typename T, int R, int E>
 int start_vec(const MixedParams& p, int tokens, int vectors, size_t smem, cudaStream_t stream) {
-  const int most = 148 * (vectors <= 6 * 256 ? 3 : 2), blocks = tokens < most ? tokens : most;  // one wave
-  if (vectors <= 2 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 2>, p, blocks, smem, stream, tokens);
-  if (vectors <= 4 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 4>, p, blocks, smem, stream, tokens);
-  if (vectors <= 6 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 6>, p, blocks, smem, stream, tokens);
-  return start(mixed_heads_prepare_vec_kernel<T, R, E, 8>, p, blocks, smem, stream, tokens);
+  if (vectors <= 3 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 3>, p, tokens, smem, stream);
+  if (vectors <= 6 * 256) return start(mixed_heads_prepare_vec_kernel<T, R, E, 6>, p, tokens, smem, stream);
+  return start(mixed_heads_prepare_vec_kernel<T, R, E, 8>, p, tokens, smem, stream);
 }
 
 template <typename T>
