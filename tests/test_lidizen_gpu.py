@@ -136,7 +136,7 @@ def test_normed_pair_embedding(dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,dim,vdim,dims,interleaved,normed", [
     (6, 3, 24, 16, 8, True, True), (4, 2, 48, 64, 48, True, True), (5, 5, 10, 12, 10, True, True), (8, 1, 128, 128, 64, True, True),
-    (8, 2, 64, 128, 0, True, False), (16, 2, 32, 32, 16, False, True), (12, 4, 16, 8, 6, False, True), (2, 2, 64, 64, 64, True, True),
+    (8, 2, 64, 128, 0, True, False), (16, 2, 32, 32, 16, False, True), (32, 4, 128, 128, 64, True, True), (16, 4, 128, 96, 126, True, True), (12, 4, 16, 8, 6, False, True), (2, 2, 64, 64, 64, True, True),
 ])  # fmt: skip
 def test_prepared_queries_keys_and_values(dtype, H, G, dim, vdim, dims, interleaved, normed):
     """Biases, the norm over the whole projection, both pairings at near and far positions, the mix of
@@ -291,7 +291,7 @@ def test_kept_positions_for_heads_that_are_not_mixed(dtype, hd, bs):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,hd,bs", [(8, 2, 128, 16), (12, 4, 64, 16), (16, 4, 128, 32), (32, 8, 64, 16), (40, 1, 64, 8), (6, 3, 40, 4), (16, 8, 128, 16),
-                                       (34, 2, 128, 16), (3, 3, 128, 64), (10, 5, 128, 16)])  # fmt: skip
+                                       (34, 2, 128, 16), (3, 3, 128, 64), (10, 5, 128, 16), (32, 8, 128, 16), (16, 16, 64, 16), (8, 8, 128, 4)])  # fmt: skip
 @pytest.mark.parametrize("window,keep", [(None, 0), (150, 70), (40, 3)])
 def test_attention_over_parts_in_mixed_batches(dtype, H, G, hd, bs, window, keep):
     """Random queries with a vector per key head: a long portion, one that starts mid-sequence, single
