@@ -204,17 +204,15 @@ parts_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
       constexpr uint32_t idesc_qk = instr_desc_bf16(kRows, kKeys, false);
       bool ok = kStreamQ || mbar_wait(q_full, 0, p.status, 12);
       const int total = num_tiles * p.KV;
-      uint32_t there = 0;  // the answer to an early question about this stage (asking takes a few hundred cycles)
       Ring ring;
       for (int n = 0, j = 0, c = 0; n < total && ok; ++n) {
         // score buffer j & 1 held tile j - 2's scores and then its P: has that tile's P V read it?
         if (c == 0 && j >= 2) ok = mbar_wait(pv_done(j & 1), ((uint32_t)(j - 2) >> 1) & 1u, p.status, 18);
         const int s = ring.stage;
-        if (ok && !there) ok = mbar_wait(k_full(s), ring.round & 1u, p.status, 13);
+        if (ok) ok = mbar_wait(k_full(s), ring.round & 1u, p.status, 13);
         if (!ok) break;
         fence_after_sync();
         ring.next(KS);
-        there = n + 1 < total ? mbar_try(k_full(ring.stage), ring.round & 1u) : 0u;
         const uint32_t q_block = kStreamQ ? k_smem(s) + kKBytes : q_smem + (uint32_t)c * kKBytes;
 #pragma unroll
         for (int ks = 0; ks < HD / 16; ++ks) {  // 16 entries per MMA: 32 bytes along the swizzled row
