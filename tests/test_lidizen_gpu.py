@@ -135,7 +135,7 @@ def test_normed_pair_embedding(dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,dim,vdim,dims,interleaved,normed", [
-    (6, 3, 24, 16, 8, True, True), (4, 2, 48, 64, 48, True, True), (5, 5, 10, 12, 10, True, True), (8, 1, 128, 128, 64, True, True),
+    (6, 3, 24, 16, 8, True, True), (8, 2, 48, 64, 40, True, True), (5, 5, 10, 12, 10, True, True), (8, 1, 128, 128, 64, True, True),
     (8, 2, 64, 128, 0, True, False), (16, 2, 32, 32, 16, False, True), (32, 4, 128, 128, 64, True, True), (16, 4, 128, 96, 126, True, True), (12, 4, 16, 8, 6, False, True), (2, 2, 64, 64, 64, True, True),
 ])  # fmt: skip
 def test_prepared_queries_keys_and_values(dtype, H, G, dim, vdim, dims, interleaved, normed):
@@ -355,7 +355,7 @@ MIXERS = [
     attention(2, 1, 8, 8, 0.5, window=1, keep=1),
     attention(3, 3, 20, 24, 0.35, window=5, rot=(30.0, 20)),
     attention(8, 2, 128, 128, 0.1, window=16, keep=6, rot=(10000.0, 64)),
-    attention(4, 2, 48, 64, 0.15, window=20, keep=20, rot=(500.0, 48)),
+    attention(8, 4, 48, 64, 0.15, window=19, keep=21, rot=(500.0, 40)),
     attention(16, 4, 64, 64, 0.12, rot=(100.0, 64)),
     attention(20, 1, 128, 96, 0.1, window=12, keep=4, rot=(100.0, 128)),
     attention(8, 8, 64, 64, 0.12, window=9, keep=2, rot=(100.0, 32)),

@@ -34,7 +34,7 @@ def model(vocab, width, streams, eps, pairs, layers):
 
 
 # sizes that only the general kernels serve
-LIDIZEN_A = model(300, 96, 3, 1e-5, (61, 31, 7), [
+LIDIZEN_A = model(300, 96, 3, 1e-5, (61, 29, 11), [
     attention(6, 3, 24, 16, 0.3, window=10, keep=3, rot=(100.0, 8), mlp=dense(72)),
     attention(4, 2, 12, 40, 0.4, window=33, keep=18, rot=(30.0, 12), v_mix=True, mlp=moe(5, 2, 40)),
     attention(2, 1, 16, 16, 0.35, rot=(1000.0, 16)),
@@ -51,7 +51,7 @@ LIDIZEN_B = model(257, 60, 1, 1e-6, (17, 3, 1000003), [
 BLOCK_SIZE_B = 8
 
 # sizes at which the bfloat16 products and attention run this package's tensor-core kernels
-LIDIZEN_C = model(704, 224, 4, 2e-6, (1021, 211, 13), [
+LIDIZEN_C = model(704, 224, 4, 2e-6, (1009, 211, 13), [
     attention(8, 2, 128, 128, 0.12, window=90, keep=30, rot=(10000.0, 64), v_mix=True, mlp=moe(8, 3, 128)),
     attention(12, 4, 64, 32, 0.16, window=64, keep=64, rot=(500.0, 64), mlp=dense(320)),
     attention(4, 2, 96, 128, 0.13, rot=(400000.0, 32), v_mix=True, mlp=moe(6, 1, 64)),
