@@ -14,14 +14,15 @@
 //                         [c | kr] to the token's cache slot; turn each head's qr and put it
 //                         behind that head's absorbed query in q_lat (float32)
 //   asb_head_matmul       out[t, h, :] = x[t, h, :] . w[h] per head (w[h]: [K, N]), optionally
-//                         times sigmoid(gate[t, h]): the query absorption and the value
-//                         up-projection with the output gate
+//                         times sigmoid(gate[t, h]) or sigmoid(gate[t, h, :]): the query absorption
+//                         and the value up-projection with the output gate
 //   asb_latent_attention  the attention itself, for any mix of prompt portions and single
 //                         tokens; float32 scores, weights and sums; key partitions aligned to
 //                         absolute positions, merged by asb_attention_reduce
 //
-// The rotation pairs neighbours: of the first `rot_dims` entries, (2i, 2i + 1) turns by
-// position * inv_freq[i]; angles are float32.
+// The rotation pairs neighbours, or halves: of the first `rot_dims` entries, (2i, 2i + 1), or
+// (i, i + rot_dims / 2), turns by position * inv_freq[i]; angles are float32. The queries may lie in a
+// tensor of their own (a low-rank query projection's second product).
 #include "common.cuh"
 
 namespace {
@@ -29,17 +30,32 @@ namespace {
 // ---- prepare ------------------------------------------------------------------------------
 
 struct PrepareParams {
-  const void* proj;        // [T, stride]
+  const void* q;           // [T, q_stride], queries from q_off on
+  const void* proj;        // [T, stride], the down-projection from kv_off on
   float* q_lat;            // [T, H, rank + rot]
   void* pages;             // [num_blocks, 1, bs, rank + rot]; null: nothing is stored
   const float* gain;       // [rank]
   const float* inv_freq;   // [rot_dims / 2]
   const int* positions;    // [T]
   const int* slots;        // [T]; negative: not stored
-  int stride, q_off, kv_off;
-  int H, D, rank, rot, rot_dims;
+  int q_stride, q_off, stride, kv_off;
+  int H, D, rank, rot, rot_dims, half_pairs;
   float eps;
 };
+
+// entry e of a vector after the rotation of its first `dims` entries
+template <typename T>
+__device__ __forceinline__ float turned_entry(const T* x, int e, int dims, int half_pairs, const float* inv_freq, float pos) {
+  const float v = asb::to_float(x[e]);
+  if (e >= dims) return v;
+  const int half = dims >> 1;
+  const bool first = half_pairs ? e < half : !(e & 1);
+  const int pair = half_pairs ? (first ? e : e - half) : e >> 1;
+  const float other = asb::to_float(x[half_pairs ? (first ? e + half : e - half) : e ^ 1]);
+  float s, c;
+  sincosf(pos * inv_freq[pair], &s, &c);
+  return first ? fmaf(v, c, -other * s) : fmaf(v, c, other * s);
+}
 
 template <typename T>
 __global__ void latent_prepare_kernel(const PrepareParams p) {
@@ -53,15 +69,8 @@ __global__ void latent_prepare_kernel(const PrepareParams p) {
   // queries: each head's turned part, behind its absorbed part
   for (int i = threadIdx.x; i < p.H * p.rot; i += blockDim.x) {
     const int h = i / p.rot, e = i - h * p.rot;
-    const T* qr = row + p.q_off + h * (p.D + p.rot) + p.D;
-    float v = asb::to_float(qr[e]);
-    if (e < p.rot_dims) {
-      float s, c;
-      sincosf(pos * p.inv_freq[e >> 1], &s, &c);
-      const float other = asb::to_float(qr[e ^ 1]);
-      v = (e & 1) ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
-    }
-    p.q_lat[((size_t)t * p.H + h) * Dk + p.rank + e] = v;
+    const T* qr = (const T*)p.q + (size_t)t * p.q_stride + p.q_off + h * (p.D + p.rot) + p.D;
+    p.q_lat[((size_t)t * p.H + h) * Dk + p.rank + e] = turned_entry(qr, e, p.rot_dims, p.half_pairs, p.inv_freq, pos);
   }
   if (!p.pages) return;
   const int slot = p.slots[t];
@@ -75,16 +84,8 @@ __global__ void latent_prepare_kernel(const PrepareParams p) {
   if (slot < 0) return;
   T* dst = (T*)p.pages + (size_t)slot * Dk;
   for (int i = threadIdx.x; i < p.rank; i += blockDim.x) dst[i] = asb::from_float<T>(asb::to_float(kv[i]) * inv * p.gain[i]);
-  for (int e = threadIdx.x; e < p.rot; e += blockDim.x) {
-    float v = asb::to_float(kv[p.rank + e]);
-    if (e < p.rot_dims) {
-      float s, c;
-      sincosf(pos * p.inv_freq[e >> 1], &s, &c);
-      const float other = asb::to_float(kv[p.rank + (e ^ 1)]);
-      v = (e & 1) ? fmaf(v, c, other * s) : fmaf(v, c, -other * s);
-    }
-    dst[p.rank + e] = asb::from_float<T>(v);
-  }
+  for (int e = threadIdx.x; e < p.rot; e += blockDim.x)
+    dst[p.rank + e] = asb::from_float<T>(turned_entry(kv + p.rank, e, p.rot_dims, p.half_pairs, p.inv_freq, pos));
 }
 
 // ---- per-head products --------------------------------------------------------------------
@@ -95,7 +96,7 @@ constexpr int kHmThreads = 128;
 template <typename TX, typename TW, typename TO>
 __global__ void __launch_bounds__(kHmThreads)
 head_matmul_kernel(TO* __restrict__ out, int out_row, int out_head, const TX* __restrict__ x, int x_row, int x_head,
-                   const TW* __restrict__ w, const TW* __restrict__ gate, int gate_row, int T, int K, int N) {
+                   const TW* __restrict__ w, const TW* __restrict__ gate, int gate_row, int gate_wide, int T, int K, int N) {
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   extern __shared__ float xs[];  // [kHmTokens][K]
@@ -120,7 +121,7 @@ head_matmul_kernel(TO* __restrict__ out, int out_row, int out_head, const TX* __
     for (int t = 0; t < kHmTokens; ++t) {
       if (t >= nt) break;
       float v = acc[t];
-      if (gate) v /= 1.f + expf(-asb::to_float(gate[(size_t)(t0 + t) * gate_row + h]));
+      if (gate) v /= 1.f + expf(-asb::to_float(gate[(size_t)(t0 + t) * gate_row + (gate_wide ? h * N + n : h)]));
       out[(size_t)(t0 + t) * out_row + (size_t)h * out_head + n] = asb::from_float<TO>(v);
     }
   }
@@ -292,13 +293,14 @@ int launch_attention(const LatentParams& p, int num_tokens, cudaStream_t stream)
 
 }  // namespace
 
-extern "C" int asb_latent_prepare(const void* proj, int stride, int q_off, int kv_off, float* q_lat, void* pages,
-                                  const float* gain, const float* inv_freq, const int* positions, const int* slots,
-                                  int T, int H, int D, int rank, int rot, int rot_dims, float eps, int dtype,
+extern "C" int asb_latent_prepare(const void* q, int q_stride, int q_off, const void* proj, int stride, int kv_off, float* q_lat,
+                                  void* pages, const float* gain, const float* inv_freq, const int* positions, const int* slots,
+                                  int T, int H, int D, int rank, int rot, int rot_dims, int half_pairs, float eps, int dtype,
                                   cudaStream_t stream) {
   if (T == 0) return 0;
   if (rot_dims % 2 || rot_dims > rot || rot_dims < 0) return asb::fail("latent_prepare: %d turned entries of %d", rot_dims, rot);
   PrepareParams p;
+  p.q = q; p.q_stride = q_stride; p.half_pairs = half_pairs;
   p.proj = proj; p.q_lat = q_lat; p.pages = pages; p.gain = gain; p.inv_freq = inv_freq;
   p.positions = positions; p.slots = slots; p.stride = stride; p.q_off = q_off; p.kv_off = kv_off;
   p.H = H; p.D = D; p.rank = rank; p.rot = rot; p.rot_dims = rot_dims; p.eps = eps;
@@ -307,10 +309,10 @@ extern "C" int asb_latent_prepare(const void* proj, int stride, int q_off, int k
 }
 
 // x: float32 (x_f32 1) or the compute dtype; out: float32 (out_f32 1) or the compute dtype; w and
-// gate in the compute dtype.
+// gate in the compute dtype; the gate holds one value a head, or (gate_wide) one per output column.
 extern "C" int asb_head_matmul(void* out, int out_f32, int out_row, int out_head, const void* x, int x_f32, int x_row,
-                               int x_head, const void* w, const void* gate, int gate_row, int T, int H, int K, int N,
-                               int dtype, cudaStream_t stream) {
+                               int x_head, const void* w, const void* gate, int gate_row, int gate_wide, int T, int H, int K,
+                               int N, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   if (H > 65535) return asb::fail("head_matmul: %d heads", H);
   const size_t smem = sizeof(float) * kHmTokens * K;
@@ -322,7 +324,7 @@ extern "C" int asb_head_matmul(void* out, int out_f32, int out_row, int out_head
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
     if (e != cudaSuccess) return asb::fail("head_matmul: shared memory %zu: %s", smem, cudaGetErrorString(e)); \
     asb::launch(kern, grid, kHmThreads, smem, stream, (TO*)out, out_row, out_head, (const TX*)x, x_row, x_head, \
-                (const TW*)w, (const TW*)gate, gate_row, T, K, N);                                             \
+                (const TW*)w, (const TW*)gate, gate_row, gate_wide, T, K, N);                                             \
   }
   ASB_DISPATCH_DTYPE(dtype, TW, {
     if (x_f32 && out_f32) ASB_HM(float, float)

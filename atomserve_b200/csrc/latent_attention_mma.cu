@@ -364,7 +364,7 @@ template <typename TX, typename TO>
 __global__ void __launch_bounds__(128)
 head_matmul_mma_kernel(TO* __restrict__ out, int out_row, int out_head, const TX* __restrict__ x, int x_row, int x_head,
                        const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __restrict__ gate, int gate_row,
-                       int T, int K, int N) {
+                       int gate_wide, int T, int K, int N) {
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   __shared__ __align__(16) __nv_bfloat16 xs[HB][HLD];
@@ -425,14 +425,17 @@ head_matmul_mma_kernel(TO* __restrict__ out, int out_row, int out_head, const TX
       const int tok = t0 + wm + i * 16 + g + half * 8;
       if (tok >= T) continue;
       float scale = 1.f;
-      if (gate) scale = 1.f / (1.f + expf(-__bfloat162float(gate[(size_t)tok * gate_row + h])));
+      if (gate && !gate_wide) scale = 1.f / (1.f + expf(-__bfloat162float(gate[(size_t)tok * gate_row + h])));
+      const __nv_bfloat16* wide = gate && gate_wide ? gate + (size_t)tok * gate_row + h * N : nullptr;
       TO* orow = out + (size_t)tok * out_row + (size_t)h * out_head;
 #pragma unroll
       for (int j = 0; j < 4; ++j)
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
           const int n = n0 + wn + j * 8 + 2 * t + c;
-          if (n < N) orow[n] = asb::from_float<TO>(acc[i][j][half * 2 + c] * scale);
+          if (n >= N) continue;
+          const float v = acc[i][j][half * 2 + c];
+          orow[n] = asb::from_float<TO>(wide ? v / (1.f + expf(-__bfloat162float(wide[n]))) : v * scale);
         }
     }
 }
@@ -443,21 +446,21 @@ extern "C" int asb_head_matmul_mma_supported(int K) { return K >= 8 && K % 8 == 
 
 // w: [H, N, K] bfloat16. x: float32 (x_f32 1) or bfloat16; out: float32 (out_f32 1) or bfloat16.
 extern "C" int asb_head_matmul_mma(void* out, int out_f32, int out_row, int out_head, const void* x, int x_f32, int x_row,
-                                   int x_head, const void* w, const void* gate, int gate_row, int T, int H, int K, int N,
-                                   cudaStream_t stream) {
+                                   int x_head, const void* w, const void* gate, int gate_row, int gate_wide, int T, int H,
+                                   int K, int N, cudaStream_t stream) {
   if (T == 0) return 0;
   if (!asb_head_matmul_mma_supported(K) || ((uintptr_t)w & 15)) return asb::fail("head_matmul_mma: K = %d must be a multiple of 8 and w 16-byte aligned", K);
   if (H > 65535 || (N + HB - 1) / HB > 65535) return asb::fail("head_matmul_mma: %d heads of %d columns exceed the grid", H, N);
   dim3 grid((T + HB - 1) / HB, H, (N + HB - 1) / HB);
   using B = __nv_bfloat16;
   if (x_f32 && out_f32)
-    asb::launch(head_matmul_mma_kernel<float, float>, grid, 128, 0, stream, (float*)out, out_row, out_head, (const float*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, T, K, N);
+    asb::launch(head_matmul_mma_kernel<float, float>, grid, 128, 0, stream, (float*)out, out_row, out_head, (const float*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, gate_wide, T, K, N);
   else if (x_f32)
-    asb::launch(head_matmul_mma_kernel<float, B>, grid, 128, 0, stream, (B*)out, out_row, out_head, (const float*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, T, K, N);
+    asb::launch(head_matmul_mma_kernel<float, B>, grid, 128, 0, stream, (B*)out, out_row, out_head, (const float*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, gate_wide, T, K, N);
   else if (out_f32)
-    asb::launch(head_matmul_mma_kernel<B, float>, grid, 128, 0, stream, (float*)out, out_row, out_head, (const B*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, T, K, N);
+    asb::launch(head_matmul_mma_kernel<B, float>, grid, 128, 0, stream, (float*)out, out_row, out_head, (const B*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, gate_wide, T, K, N);
   else
-    asb::launch(head_matmul_mma_kernel<B, B>, grid, 128, 0, stream, (B*)out, out_row, out_head, (const B*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, T, K, N);
+    asb::launch(head_matmul_mma_kernel<B, B>, grid, 128, 0, stream, (B*)out, out_row, out_head, (const B*)x, x_row, x_head, (const B*)w, (const B*)gate, gate_row, gate_wide, T, K, N);
   return asb::check_launch("head_matmul_mma");
 }
 

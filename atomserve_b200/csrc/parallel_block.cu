@@ -2,10 +2,10 @@
 // x <- x + mult (mixer(N1 x) + ff(N2 x)), over a float32 residual stream, and for what such a
 // model does around its layers:
 //
-//   asb_residual_dual_norm   s = x + mult (y1 + y2) + bias (every term optional), written as the
-//                            float32 stream, and N(s) gain1, N(s) gain2 in the compute dtype,
-//                            N(s) = s / sqrt(mean(s^2) + eps): the sum of a layer and both norms of
-//                            the next one in one pass over the row
+//   asb_residual_terms_norm  s = x + sum_i f_i y_i + bias (up to four terms, x and bias optional),
+//                            written as the float32 stream, and N(s) gain1, N(s) gain2 in the compute
+//                            dtype, N(s) = s / sqrt(mean(s^2) + eps): the sum of a layer, whatever
+//                            number of outputs it has, and both norms of the next one in one pass
 //   asb_pair_embedding       x[t] = table[id[t]] + pairs[row(previous id, id[t])], float32: a
 //                            hashed table of token pairs beside the token table. The id before a
 //                            request's first token of the step is per-request state (0: none yet)
@@ -23,13 +23,18 @@ int threads_for(int width) {
   return threads;
 }
 
+constexpr int kMaxTerms = 4;
+struct Terms {
+  const float* y[kMaxTerms];
+  float f[kMaxTerms];
+  int n;
+};
+
 // One block per row; the row's sum stays in shared memory between the two passes.
 template <typename T>
-__global__ void residual_dual_norm_kernel(float* __restrict__ out32, T* __restrict__ out1, T* __restrict__ out2,
-                                          const float* __restrict__ x, const float* __restrict__ y1,
-                                          const float* __restrict__ y2, const float* __restrict__ bias,
-                                          const float* __restrict__ gain1, const float* __restrict__ gain2,
-                                          int width, float mult, float eps) {
+__global__ void residual_terms_norm_kernel(float* __restrict__ out32, T* __restrict__ out1, T* __restrict__ out2,
+                                           const float* __restrict__ x, const Terms terms, const float* __restrict__ bias,
+                                           const float* __restrict__ gain1, const float* __restrict__ gain2, int width, float eps) {
   extern __shared__ float row[];
   __shared__ float scratch[32];
   asb::pdl_wait();
@@ -37,9 +42,10 @@ __global__ void residual_dual_norm_kernel(float* __restrict__ out32, T* __restri
   const size_t at = (size_t)blockIdx.x * width;
   float ss = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
-    float y = y1 ? y1[at + i] : 0.f;
-    if (y2) y += y2[at + i];
-    float s = x ? fmaf(mult, y, x[at + i]) : mult * y;
+    float s = x ? x[at + i] : 0.f;
+#pragma unroll
+    for (int u = 0; u < kMaxTerms; ++u)
+      if (u < terms.n) s = fmaf(terms.f[u], terms.y[u][at + i], s);
     if (bias) s += bias[i];
     row[i] = s;
     ss = fmaf(s, s, ss);
@@ -51,6 +57,74 @@ __global__ void residual_dual_norm_kernel(float* __restrict__ out32, T* __restri
     const float n = s * inv;
     if (out1) out1[at + i] = asb::from_float<T>(n * gain1[i]);
     if (out2) out2[at + i] = asb::from_float<T>(n * gain2[i]);
+  }
+}
+
+__device__ __forceinline__ void store4(float* at, float4 v) { *reinterpret_cast<float4*>(at) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* at, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(at) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
+// The same where rows are whole vectors of four: a thread keeps its NV vectors in registers, all loads of a
+// term in flight together.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+residual_terms_norm_vec_kernel(float* __restrict__ out32, T* __restrict__ out1, T* __restrict__ out2, const float* __restrict__ x,
+                               const Terms terms, const float* __restrict__ bias, const float* __restrict__ gain1,
+                               const float* __restrict__ gain2, int width, float eps) {
+  __shared__ float scratch[32];
+  asb::pdl_wait();
+  asb::pdl_launch_dependents();
+  const size_t at = (size_t)blockIdx.x * width;
+  float4 s[NV];
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (threadIdx.x + v * blockDim.x) * 4;
+    s[v] = (x && i < width) ? *reinterpret_cast<const float4*>(x + at + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int u = 0; u < kMaxTerms; ++u) {
+    if (u >= terms.n) break;
+    const float f = terms.f[u];
+    float4 y[NV];
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int i = (threadIdx.x + v * blockDim.x) * 4;
+      y[v] = i < width ? *reinterpret_cast<const float4*>(terms.y[u] + at + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      s[v].x = fmaf(f, y[v].x, s[v].x); s[v].y = fmaf(f, y[v].y, s[v].y);
+      s[v].z = fmaf(f, y[v].z, s[v].z); s[v].w = fmaf(f, y[v].w, s[v].w);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (threadIdx.x + v * blockDim.x) * 4;
+    if (bias && i < width) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + i);
+      s[v].x += b.x; s[v].y += b.y; s[v].z += b.z; s[v].w += b.w;
+    }
+    ss = fmaf(s[v].x, s[v].x, fmaf(s[v].y, s[v].y, fmaf(s[v].z, s[v].z, fmaf(s[v].w, s[v].w, ss))));
+  }
+  float inv = 0.f;
+  if (out1 || out2) inv = 1.f / sqrtf(asb::block_sum(ss, scratch) / (float)width + eps);
+#pragma unroll
+  for (int v = 0; v < NV; ++v) {
+    const int i = (threadIdx.x + v * blockDim.x) * 4;
+    if (i >= width) break;
+    if (out32) store4(out32 + at + i, s[v]);
+    const float4 n = make_float4(s[v].x * inv, s[v].y * inv, s[v].z * inv, s[v].w * inv);
+    if (out1) {
+      const float4 g = *reinterpret_cast<const float4*>(gain1 + i);
+      store4(out1 + at + i, make_float4(n.x * g.x, n.y * g.y, n.z * g.z, n.w * g.w));
+    }
+    if (out2) {
+      const float4 g = *reinterpret_cast<const float4*>(gain2 + i);
+      store4(out2 + at + i, make_float4(n.x * g.x, n.y * g.y, n.z * g.z, n.w * g.w));
+    }
   }
 }
 
@@ -147,17 +221,38 @@ __global__ void concat_cast_kernel(T* __restrict__ out, const float* __restrict_
 
 }  // namespace
 
-// out32, out1, out2, x, y1, y2, bias: each may be null (out2 with gain2). dtype is that of out1/out2.
-extern "C" int asb_residual_dual_norm(float* out32, void* out1, void* out2, const float* x, const float* y1,
-                                      const float* y2, const float* bias, const float* gain1, const float* gain2,
-                                      int n, int width, float mult, float eps, int dtype, cudaStream_t stream) {
+// out32, out1, out2, x, bias: each may be null (out1 with gain1, out2 with gain2); y1 .. y4 with their factors:
+// the first `terms` of them. dtype is that of out1 and out2.
+extern "C" int asb_residual_terms_norm(float* out32, void* out1, void* out2, const float* x, const float* y1, const float* y2,
+                                       const float* y3, const float* y4, float f1, float f2, float f3, float f4, int terms,
+                                       const float* bias, const float* gain1, const float* gain2, int n, int width, float eps,
+                                       int dtype, cudaStream_t stream) {
   if (n == 0) return 0;
-  if (width < 1 || width > 48 * 1024 / 4) return asb::fail("residual_dual_norm: width %d not in 1..12288", width);
-  if ((out1 && !gain1) || (out2 && !gain2)) return asb::fail("residual_dual_norm: a normed output needs its gain");
-  ASB_DISPATCH_DTYPE(dtype, T, asb::launch(residual_dual_norm_kernel<T>, n, threads_for(width), width * sizeof(float),
-                                           stream, out32, (T*)out1, (T*)out2, x, y1, y2, bias, gain1, gain2, width,
-                                           mult, eps));
-  return asb::check_launch("residual_dual_norm");
+  if (width < 1 || width > 48 * 1024 / 4) return asb::fail("residual_terms_norm: width %d not in 1..12288", width);
+  if (terms < 0 || terms > kMaxTerms) return asb::fail("residual_terms_norm: %d terms, at most %d", terms, kMaxTerms);
+  if ((out1 && !gain1) || (out2 && !gain2)) return asb::fail("residual_terms_norm: a normed output needs its gain");
+  const Terms t = {{y1, y2, y3, y4}, {f1, f2, f3, f4}, terms};
+  uintptr_t all = (uintptr_t)out32 | (uintptr_t)out1 | (uintptr_t)out2 | (uintptr_t)x | (uintptr_t)bias | (uintptr_t)gain1 | (uintptr_t)gain2;
+  for (int u = 0; u < terms; ++u) {
+    if (!t.y[u]) return asb::fail("residual_terms_norm: term %d is missing", u);
+    all |= (uintptr_t)t.y[u];
+  }
+  if (width % 4 == 0 && width <= 8192 && (all & 15) == 0) {
+    const int vectors = width / 4, nv = vectors <= 256 ? 1 : (vectors <= 512 ? 2 : (vectors <= 1024 ? 4 : 8));
+    const int threads = ((vectors + nv - 1) / nv + 31) / 32 * 32;
+#define ASB_TERMS(NV)                                                                                                     \
+  ASB_DISPATCH_DTYPE(dtype, T, asb::launch(residual_terms_norm_vec_kernel<T, NV>, n, threads, 0, stream, out32, (T*)out1, \
+                                           (T*)out2, x, t, bias, gain1, gain2, width, eps))
+    if (nv == 1) ASB_TERMS(1);
+    else if (nv == 2) ASB_TERMS(2);
+    else if (nv == 4) ASB_TERMS(4);
+    else ASB_TERMS(8);
+#undef ASB_TERMS
+    return asb::check_launch("residual_terms_norm");
+  }
+  ASB_DISPATCH_DTYPE(dtype, T, asb::launch(residual_terms_norm_kernel<T>, n, threads_for(width), width * sizeof(float),
+                                           stream, out32, (T*)out1, (T*)out2, x, t, bias, gain1, gain2, width, eps));
+  return asb::check_launch("residual_terms_norm");
 }
 
 extern "C" int asb_pair_embedding(float* out, const void* table, const void* pairs, const int* ids,

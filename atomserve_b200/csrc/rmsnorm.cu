@@ -13,12 +13,12 @@ namespace {
 template <typename T>
 __global__ void rmsnorm_kernel(T* __restrict__ out, const T* __restrict__ x,
                                const float* __restrict__ gain, const int* __restrict__ rows,
-                               int width, float eps) {
+                               int width, int x_stride, float eps) {
   asb::pdl_wait();  // the stream's previous kernel has completed (programmatic dependent launch)
   asb::pdl_launch_dependents();
   __shared__ float scratch[32];
   const int r = blockIdx.x;
-  const T* src = x + (size_t)(rows ? rows[r] : r) * width;
+  const T* src = x + (size_t)(rows ? rows[r] : r) * x_stride;
   T* dst = out + (size_t)r * width;
   float ss = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
@@ -36,12 +36,12 @@ __global__ void rmsnorm_kernel(T* __restrict__ out, const T* __restrict__ x,
 template <typename T, int VEC>
 __global__ void rmsnorm_vec_kernel(T* __restrict__ out, const T* __restrict__ x,
                                    const float* __restrict__ gain, const int* __restrict__ rows,
-                                   int width, float eps) {
+                                   int width, int x_stride, float eps) {
   asb::pdl_wait();  // the stream's previous kernel has completed (programmatic dependent launch)
   asb::pdl_launch_dependents();
   __shared__ float scratch[32];
   const int r = blockIdx.x;
-  const T* src = x + (size_t)(rows ? rows[r] : r) * width;
+  const T* src = x + (size_t)(rows ? rows[r] : r) * x_stride;
   T* dst = out + (size_t)r * width;
   const int i = threadIdx.x * VEC;
   const bool active = i < width;
@@ -126,27 +126,28 @@ __global__ void partial_add_rmsnorm_kernel(__nv_bfloat16* __restrict__ sum_out, 
 }
 
 template <typename T>
-int launch(void* out, const void* x, const float* gain, const int* rows, int num_rows, int width,
+int launch(void* out, const void* x, int x_stride, const float* gain, const int* rows, int num_rows, int width,
            float eps, cudaStream_t stream) {
   constexpr int VEC = 16 / sizeof(T);
   const bool aligned = ((uintptr_t)out % 16 == 0) && ((uintptr_t)x % 16 == 0) && ((uintptr_t)gain % 16 == 0);
-  if (width % VEC == 0 && width / VEC <= 1024 && aligned) {
+  if (width % VEC == 0 && x_stride % VEC == 0 && width / VEC <= 1024 && aligned) {
     const int threads = ((width / VEC) + 31) / 32 * 32;
-    asb::launch(rmsnorm_vec_kernel<T, VEC>, num_rows, threads, 0, stream, (T*)out, (const T*)x, gain, rows, width, eps);
+    asb::launch(rmsnorm_vec_kernel<T, VEC>, num_rows, threads, 0, stream, (T*)out, (const T*)x, gain, rows, width, x_stride, eps);
   } else {
     int threads = 32;
     while (threads < 1024 && threads * 4 < width) threads <<= 1;
-    asb::launch(rmsnorm_kernel<T>, num_rows, threads, 0, stream, (T*)out, (const T*)x, gain, rows, width, eps);
+    asb::launch(rmsnorm_kernel<T>, num_rows, threads, 0, stream, (T*)out, (const T*)x, gain, rows, width, x_stride, eps);
   }
   return asb::check_launch("rmsnorm");
 }
 
 }  // namespace
 
-extern "C" int asb_rmsnorm(void* out, const void* x, const float* gain, const int* rows,
+// x: rows of x_stride elements, of which the first `width` are normed.
+extern "C" int asb_rmsnorm(void* out, const void* x, int x_stride, const float* gain, const int* rows,
                            int num_rows, int width, float eps, int dtype, cudaStream_t stream) {
   if (num_rows == 0) return 0;
-  ASB_DISPATCH_DTYPE(dtype, T, return launch<T>(out, x, gain, rows, num_rows, width, eps, stream));
+  ASB_DISPATCH_DTYPE(dtype, T, return launch<T>(out, x, x_stride, gain, rows, num_rows, width, eps, stream));
   return 0;
 }
 

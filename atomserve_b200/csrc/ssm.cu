@@ -8,9 +8,13 @@
 //                          inputs before a portion's first token read from the request's state
 //                          (the last K - 1 inputs of what came before; zeros for a new request).
 //                          In the same launch, per head: dt = softplus(z + dt_bias_h), the token's
-//                          decay exp(-exp(A_h) dt) and input weight dt, all float32.
+//                          decay exp(-exp(A_h) dt) and input weight dt, all float32. The bias and the
+//                          step columns are optional. Requests that bring at most one tile of tokens
+//                          (decoded tokens, short portions) can have their state updated in the same
+//                          launch: every channel of theirs is one thread's.
 //   asb_conv_state_update  the state after the step: the last K - 1 inputs of each request
-//                          (a portion shorter than that shifts what the state held).
+//                          (a portion shorter than that shifts what the state held); requests of at
+//                          most `skip` tokens are left alone.
 //   asb_gate_group_norm    (y + D_h x) silu(z), RMS-normed in equal parts of the row (each part by
 //                          its own root mean square), times a gain: the gate comes before the norm.
 //
@@ -33,13 +37,14 @@ struct ConvParams {
   float* weight;           // [T, H]
   const void* proj;        // [T, stride]
   const float* taps;       // [C, K]
-  const float* bias;       // [C]
-  const float* conv_state; // [slots, K - 1, C]
+  const float* bias;       // [C] or null
+  float* conv_state;       // [slots, K - 1, C]
   const float* dt_bias;    // [H]
   const float* a_log;      // [H]
   const int* state_slots;  // [R]
   const int* req_q_start;  // [R + 1]
   int stride, conv_off, dt_off, C, K, H, R;
+  int update;              // 1: requests of one tile have their state updated here
 };
 
 // V neighbouring channels of one token in one load or store (V = 2 where every row's channels start at an
@@ -65,6 +70,20 @@ template <> struct Lanes<float, 2> {
   }
   static __device__ __forceinline__ void store(float* at, const float* v) { *reinterpret_cast<float2*>(at) = make_float2(v[0], v[1]); }
 };
+
+// The state after a request's n tokens, for V channels that no other thread touches: entry s of the new
+// state is input n - (K - 1) + s of the portion; a negative index is what the old state held at s + n (read
+// before any entry at or above it is written: s rises).
+template <typename T, int V>
+__device__ __forceinline__ void keep_last_inputs(float* held, const T* in, size_t stride, int n, int K, int C) {
+  for (int s = 0; s < K - 1; ++s) {
+    const int at = n - (K - 1) + s;
+    float v[V];
+    if (at >= 0) Lanes<T, V>::load(in + (size_t)at * stride, v);
+    else Lanes<float, V>::load(held + (size_t)(s + n) * C, v);
+    Lanes<float, V>::store(held + (size_t)s * C, v);
+  }
+}
 
 // grid.x: token tiles of all requests (a block finds its request by bisection), grid.y: chunks of 128
 // columns: the C / V groups of V neighbouring channels, then the H step columns.
@@ -102,12 +121,12 @@ conv_steps_kernel(const ConvParams p) {
   }
   const int K = p.K, c = column * V;
   const float* w = p.taps + (size_t)c * K;  // channel c + v's taps: w[v * K ..]
-  const float* held = p.conv_state + (size_t)p.state_slots[r] * (K - 1) * p.C + c;
+  float* held = p.conv_state + (size_t)p.state_slots[r] * (K - 1) * p.C + c;
   const T* in = proj + p.conv_off + c;
   T* out = (T*)p.out;
   float b[V];
 #pragma unroll
-  for (int v = 0; v < V; ++v) b[v] = p.bias[c + v];
+  for (int v = 0; v < V; ++v) b[v] = p.bias ? p.bias[c + v] : 0.f;
   if (K <= kConvWindow) {
     // Up to kConvWindow taps: the taps padded in front with zeros to kConvWindow (a zero tap leaves the
     // sum as it is, so the sum runs in the same order as below), the last kConvWindow - 1 inputs kept in
@@ -162,6 +181,7 @@ conv_steps_kernel(const ConvParams p) {
 #pragma unroll
         for (int v = 0; v < V; ++v) hist[i][v] = x[kConvWindow + i][v];
     }
+    if (p.update && q_len <= kConvTokens) keep_last_inputs<T, V>(held, in + (size_t)row_lo * p.stride, p.stride, q_len, K, p.C);
     return;
   }
   for (int v = 0; v < V; ++v) {
@@ -175,23 +195,20 @@ conv_steps_kernel(const ConvParams p) {
       out[(size_t)(row_lo + q) * p.C + c + v] = asb::from_float<T>(silu_f(acc));
     }
   }
+  if (p.update && q_len <= kConvTokens) keep_last_inputs<T, V>(held, in + (size_t)row_lo * p.stride, p.stride, q_len, K, p.C);
 }
 
 template <typename T>
 __global__ void conv_state_update_kernel(float* __restrict__ conv_state, const T* __restrict__ proj, int stride, int conv_off,
-                                         const int* __restrict__ state_slots, const int* __restrict__ req_q_start, int C, int K) {
+                                         const int* __restrict__ state_slots, const int* __restrict__ req_q_start, int C, int K, int skip) {
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   const int r = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= C) return;
   const int row_lo = req_q_start[r], n = req_q_start[r + 1] - row_lo;
-  float* held = conv_state + (size_t)state_slots[r] * (K - 1) * C + c;
-  // entry s of the new state is input n - (K - 1) + s of the portion; a negative index is what the old
-  // state held at s + n (read before any entry at or above it is written: s rises)
-  for (int s = 0; s < K - 1; ++s) {
-    const int at = n - (K - 1) + s;
-    held[(size_t)s * C] = at >= 0 ? asb::to_float(proj[(size_t)(row_lo + at) * stride + conv_off + c]) : held[(size_t)(s + n) * C];
-  }
+  if (n <= skip) return;
+  keep_last_inputs<T, 1>(conv_state + (size_t)state_slots[r] * (K - 1) * C + c, proj + (size_t)row_lo * stride + conv_off + c,
+                         stride, n, K, C);
 }
 
 // One block per (token, part of the row).
@@ -223,16 +240,20 @@ __global__ void gate_group_norm_kernel(T* __restrict__ out, const float* __restr
 
 }  // namespace
 
+// Tokens up to which asb_conv_steps with `update` leaves a request's state as the step ends.
+extern "C" int asb_conv_tile_tokens() { return kConvTokens; }
+
 extern "C" int asb_conv_steps(void* out, float* decay, float* weight, const void* proj, int stride, int conv_off, int dt_off,
-                              const float* taps, const float* bias, const float* conv_state, const float* dt_bias,
+                              const float* taps, const float* bias, float* conv_state, const float* dt_bias,
                               const float* a_log, const int* state_slots, const int* req_q_start, int num_tokens, int R,
-                              int C, int K, int H, int dtype, cudaStream_t stream) {
+                              int C, int K, int H, int update, int dtype, cudaStream_t stream) {
   if (num_tokens == 0 || R == 0) return 0;
   if (K < 1 || K > 64) return asb::fail("conv_steps: %d taps", K);
   ConvParams p;
   p.out = out; p.decay = decay; p.weight = weight; p.proj = proj; p.taps = taps; p.bias = bias; p.conv_state = conv_state;
   p.dt_bias = dt_bias; p.a_log = a_log; p.state_slots = state_slots; p.req_q_start = req_q_start;
   p.stride = stride; p.conv_off = conv_off; p.dt_off = dt_off; p.C = C; p.K = K; p.H = H; p.R = R;
+  p.update = update;
   // two channels a thread where every row's channels start at an even element (and so at 4 or 8 bytes)
   const int esize = dtype == asb::kFloat32 ? 4 : 2;
   const bool two = C % 2 == 0 && conv_off % 2 == 0 && stride % 2 == 0 && K <= kConvWindow &&
@@ -248,11 +269,11 @@ extern "C" int asb_conv_steps(void* out, float* decay, float* weight, const void
 }
 
 extern "C" int asb_conv_state_update(float* conv_state, const void* proj, int stride, int conv_off, const int* state_slots,
-                                     const int* req_q_start, int R, int C, int K, int dtype, cudaStream_t stream) {
+                                     const int* req_q_start, int R, int C, int K, int skip, int dtype, cudaStream_t stream) {
   if (R == 0 || K < 2) return 0;
   dim3 grid(R, (C + 127) / 128);
   ASB_DISPATCH_DTYPE(dtype, T, asb::launch(conv_state_update_kernel<T>, grid, 128, 0, stream, conv_state, (const T*)proj,
-                                           stride, conv_off, state_slots, req_q_start, C, K));
+                                           stride, conv_off, state_slots, req_q_start, C, K, skip));
   return asb::check_launch("conv_state_update");
 }
 

@@ -33,18 +33,19 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, status: torch.Tensor) -> t
 
 
 def rms_norm(x: torch.Tensor, gain: torch.Tensor, eps: float, rows: torch.Tensor | None = None) -> torch.Tensor:
-    """gain * x / sqrt(mean(x^2) + eps) over the last dim of x [N, d]; with `rows` (int32 [n])
-    only those rows of x are normalised and returned, in that order."""
+    """gain * x / sqrt(mean(x^2) + eps) over the last dim of x [N, d] (rows may be strided: a column
+    range of a projection); with `rows` (int32 [n]) only those rows of x are normalised and returned,
+    in that order."""
     require_cuda(x, gain, rows)
-    if x.dim() != 2 or not x.is_contiguous():
-        raise KernelLibraryError("rms_norm takes a contiguous [rows, width] tensor")
+    if x.dim() != 2 or x.stride(1) != 1:
+        raise KernelLibraryError("rms_norm takes a [rows, width] tensor with unit column stride")
     _gain(gain, x.shape[1], "gain")
     n = x.shape[0]
     if rows is not None:
         _int32(rows, "rows")
         n = rows.shape[0]
     out = torch.empty(n, x.shape[1], device=x.device, dtype=x.dtype)
-    check(lib().asb_rmsnorm(ptr(out), ptr(x), ptr(gain), ptr(rows), n, x.shape[1], float(eps),
+    check(lib().asb_rmsnorm(ptr(out), ptr(x), x.stride(0), ptr(gain), ptr(rows), n, x.shape[1], float(eps),
                             dtype_code(x), stream()))  # fmt: skip
     return out
 

@@ -20,13 +20,18 @@ ATTENTION_KERNEL = os.environ.get("ATOMSERVE_B200_LATENT_ATTENTION", "mma")
 def latent_prepare(proj: torch.Tensor, q_off: int, kv_off: int | None, q_lat: torch.Tensor, pages: torch.Tensor | None,
                    gain: torch.Tensor | None, inv_freq: torch.Tensor | None, positions: torch.Tensor,
                    slots: torch.Tensor | None, *, heads: int, dim: int, rank: int, rot: int, rot_dims: int,
-                   eps: float) -> None:  # fmt: skip
+                   eps: float, queries: torch.Tensor | None = None, half_pairs: bool = False) -> None:  # fmt: skip
     """Per token of proj [T, W]: with `pages` ([num_blocks, 1, block_size, rank + rot]), write
     [rms_norm(latent) * gain | turned shared key part] to the token's slot, the latent being the
     `rank` columns from kv_off and the key part the `rot` after them; and turn the last `rot` of
     each head's dim + rot query columns (from q_off) into q_lat[t, h, rank:] (float32). Of the
-    `rot` entries the first `rot_dims` turn, neighbours paired (rot 0: no such part, no frequencies)."""
-    require_cuda(proj, q_lat, pages, gain, inv_freq, positions, slots)
+    `rot` entries the first `rot_dims` turn, neighbours paired, or with `half_pairs` entry i with
+    i + rot_dims / 2 (rot 0: no such part, no frequencies). `queries`, where the queries lie in a tensor
+    of their own ([T, columns], from q_off there)."""
+    require_cuda(proj, q_lat, pages, gain, inv_freq, positions, slots, queries)
+    q = proj if queries is None else queries
+    if q.dim() != 2 or not q.is_contiguous() or q.dtype != proj.dtype or q.shape[0] != proj.shape[0] or q_off + heads * (dim + rot) > q.shape[1]:
+        raise KernelLibraryError("latent_prepare: queries must be a contiguous [tokens, columns] tensor in proj's dtype")
     if proj.dim() != 2 or not proj.is_contiguous():
         raise KernelLibraryError("latent_prepare: proj must be a contiguous [tokens, columns] tensor")
     T = proj.shape[0]
@@ -39,9 +44,9 @@ def latent_prepare(proj: torch.Tensor, q_off: int, kv_off: int | None, q_lat: to
             raise KernelLibraryError("latent_prepare: pages must be [num_blocks, 1, block_size, rank + rot] in proj's dtype")
         if gain is None or gain.dtype != torch.float32 or gain.shape != (rank,) or slots is None or kv_off is None:
             raise KernelLibraryError("latent_prepare: storing needs the latent's gain, its columns and the slots")
-    check(lib().asb_latent_prepare(ptr(proj), proj.shape[1], q_off, kv_off or 0, ptr(q_lat), ptr(pages), ptr(gain),
+    check(lib().asb_latent_prepare(ptr(q), q.shape[1], q_off, ptr(proj), proj.shape[1], kv_off or 0, ptr(q_lat), ptr(pages), ptr(gain),
                                    ptr(inv_freq), ptr(positions), ptr(slots), T, heads, dim, rank, rot, rot_dims,
-                                   float(eps), dtype_code(proj), stream()))  # fmt: skip
+                                   int(half_pairs), float(eps), dtype_code(proj), stream()))  # fmt: skip
 
 
 def head_matmul_on_tensor_cores(w: torch.Tensor, k: int) -> bool:
@@ -52,7 +57,8 @@ def head_matmul_on_tensor_cores(w: torch.Tensor, k: int) -> bool:
 
 def head_matmul(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None,
                 w_is_nk: bool = False) -> torch.Tensor:  # fmt: skip
-    """out[t, h, :] = x[t, h, :] . w[h], times sigmoid(gate[t, h]) where a gate is given. w is
+    """out[t, h, :] = x[t, h, :] . w[h], times sigmoid(gate) where a gate is given: [T, H], one value a
+    head, or [T, H * N], one per output column. w is
     [H, K, N] in the compute dtype, or with `w_is_nk` [H, N, K] in bfloat16 (the tensor-core
     kernel's layout). x [T, H, K] and out [T, H, N] are float32 or the compute dtype and may be
     strided views with unit stride along the last axis."""
@@ -64,18 +70,19 @@ def head_matmul(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: torch
     for t in (x, out):
         if t.dtype not in (torch.float32, w.dtype):
             raise KernelLibraryError("head_matmul: x and out are float32 or w's dtype")
-    if gate is not None and (gate.shape != (T, H) or gate.dtype != w.dtype or gate.stride(1) != 1):
-        raise KernelLibraryError("head_matmul: gate must be [T, H] in w's dtype with unit column stride")
+    wide = gate is not None and gate.shape == (T, H * N) and N > 1
+    if gate is not None and ((gate.shape != (T, H) and not wide) or gate.dtype != w.dtype or gate.stride(1) != 1):
+        raise KernelLibraryError("head_matmul: gate must be [T, H] or [T, H * N] in w's dtype with unit column stride")
     if w_is_nk:
         if not head_matmul_on_tensor_cores(w, K) or w.data_ptr() % 16:
             raise KernelLibraryError("head_matmul: [H, N, K] weights are bfloat16 with K a multiple of 8")
         check(lib().asb_head_matmul_mma(ptr(out), int(out.dtype == torch.float32), out.stride(0), out.stride(1), ptr(x),
                                         int(x.dtype == torch.float32), x.stride(0), x.stride(1), ptr(w), ptr(gate),
-                                        gate.stride(0) if gate is not None else 0, T, H, K, N, stream()))  # fmt: skip
+                                        gate.stride(0) if gate is not None else 0, int(wide), T, H, K, N, stream()))  # fmt: skip
         return out
     check(lib().asb_head_matmul(ptr(out), int(out.dtype == torch.float32), out.stride(0), out.stride(1), ptr(x),
                                 int(x.dtype == torch.float32), x.stride(0), x.stride(1), ptr(w), ptr(gate),
-                                gate.stride(0) if gate is not None else 0, T, H, K, N, dtype_code(w), stream()))  # fmt: skip
+                                gate.stride(0) if gate is not None else 0, int(wide), T, H, K, N, dtype_code(w), stream()))  # fmt: skip
     return out
 
 

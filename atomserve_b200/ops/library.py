@@ -28,7 +28,7 @@ class KernelLibraryError(RuntimeError):
 _P, _I, _F = c_void_p, c_int, c_float
 _SIGNATURES = {
     "asb_embedding": [_P, _P, _P, _I, _I, _I, _I, _P, _P],
-    "asb_rmsnorm": [_P, _P, _P, _P, _I, _I, _F, _I, _P],
+    "asb_rmsnorm": [_P, _P, _I, _P, _P, _I, _I, _F, _I, _P],
     "asb_silu_mul": [_P, _P, _I, _I, _I, _P],
     "asb_qk_norm_rope_store": [_P] * 9 + [_I] * 6 + [_F, _I, _P],
     "asb_paged_attention": [_P] * 10 + [_I] * 10 + [_F, _I, _P],
@@ -64,8 +64,9 @@ _SIGNATURES = {
     "asb_linear_recurrence_shared": [_P, _P, _I, _I, _I, _I] + [_P] * 10 + [_I, _F, _F] + [_I] * 8 + [_P],
     "asb_rotary_table": [_P, _P, _P, _I, _I, _P],
     # a state-space recurrence's convolution, step sizes and gated norm
-    "asb_conv_steps": [_P, _P, _P, _P, _I, _I, _I] + [_P] * 7 + [_I] * 6 + [_P],
-    "asb_conv_state_update": [_P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _P],
+    "asb_conv_steps": [_P, _P, _P, _P, _I, _I, _I] + [_P] * 7 + [_I] * 7 + [_P],
+    "asb_conv_tile_tokens": [],
+    "asb_conv_state_update": [_P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     "asb_gate_group_norm": [_P, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P],
     # blocks with a norm on a sublayer's input and on its output
     "asb_add_normed": [_P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _F, _F, _I, _P],
@@ -84,12 +85,12 @@ _SIGNATURES = {
     "asb_capped_gates_scan": [_P, _P, _P, _P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _I, _F, _P],
     "asb_gated_token_slice": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     # attention over a cached latent
-    "asb_latent_prepare": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P],
-    "asb_head_matmul": [_P, _I, _I, _I, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "asb_latent_prepare": [_P, _I, _I, _P, _I, _I] + [_P] * 6 + [_I] * 7 + [_F, _I, _P],
+    "asb_head_matmul": [_P, _I, _I, _I, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "asb_latent_attention": [_P] * 9 + [_I] * 9 + [_F, _I, _I, _P],
     "asb_latent_attention_mma": [_P] * 9 + [_I] * 9 + [_F, _I, _P],
     "asb_latent_attention_mma_supported": [_I, _I],
-    "asb_head_matmul_mma": [_P, _I, _I, _I, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+    "asb_head_matmul_mma": [_P, _I, _I, _I, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     # routed experts
     "asb_moe_route": [_P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _P],
     "asb_moe_group": [_P, _I, _I, _I, _P, _P, _P, _P],
@@ -105,7 +106,7 @@ _SIGNATURES = {
     "asb_paged_attention_mma_masked": [_P] * 11 + [_I] * 11 + [_F, _F, _I, _I, _I, _I, _P],
     "asb_prefill_attention_tcgen05_masked": [_P] * 8 + [_I] * 10 + [_F, _F, _P, _P],
     # layers whose two sublayers read one stream; a hashed table of token pairs; a product over two streams
-    "asb_residual_dual_norm": [_P] * 9 + [_I, _I, _F, _F, _I, _P],
+    "asb_residual_terms_norm": [_P] * 8 + [_F] * 4 + [_I] + [_P] * 3 + [_I, _I, _F, _I, _P],
     "asb_pair_embedding": [_P] * 8 + [_I] * 8 + [_P, _P],
     "asb_concat_cast": [_P, _P, _P, _I, _I, _I, _P],
     # parallel residual streams; scores mixed across heads, kept first positions; experts without a gate
@@ -120,6 +121,11 @@ _SIGNATURES = {
     "asb_attention_parts_resident": [_I, _I, _I],
     "asb_moe_relu2": [_P] * 5 + [_I] * 5 + [_P],
     "asb_moe_relu2_mma": [_P] * 5 + [_I] * 4 + [_P],
+    # the gated delta rule; queries and keys normed over their whole projection and turned
+    "asb_delta_chunk_tokens": [_I],
+    "asb_delta_step": [_P, _P] + [_I] * 4 + [_P] + [_I] * 3 + [_P] * 5 + [_I] * 5 + [_F, _I, _I, _P],
+    "asb_delta_chunks": [_P, _P] + [_I] * 4 + [_P] + [_I] * 3 + [_P] * 12 + [_I] * 6 + [_F, _I, _P],
+    "asb_projection_norm_rope_store": [_P, _I, _I] + [_P] * 8 + [_I] * 9 + [_F, _I, _P],
     # heads of several score maps
     "asb_qk_prepare_store": [_P] * 7 + [_I] * 10 + [_F, _I, _I, _P],
     "asb_differential_combine": [_P, _P, _I, _I, _I, _F, _F, _F, _I, _P],

@@ -14,29 +14,40 @@ def _rows32(t: torch.Tensor | None, name: str, shape: tuple) -> None:
         raise KernelLibraryError(f"{name} must be contiguous float32 {list(shape)}, got {t.dtype} {tuple(t.shape)}")
 
 
-def residual_dual_norm(x: torch.Tensor | None, y1: torch.Tensor | None, y2: torch.Tensor | None, mult: float,
-                       gain1: torch.Tensor | None, gain2: torch.Tensor | None, eps: float, dtype: torch.dtype, *,
-                       bias: torch.Tensor | None = None,
-                       want_stream: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None, torch.Tensor | None]:  # fmt: skip
-    """s = x + mult (y1 + y2) + bias, every term optional (float32 [n, width]; bias [width]), and
-    its two norms N(s) gain1, N(s) gain2 in `dtype`, N(s) = s / sqrt(mean(s^2) + eps). Returns
-    (s or None, first norm or None, second norm or None)."""
-    first = next((t for t in (x, y1, y2) if t is not None), None)
-    if first is None:
-        raise KernelLibraryError("residual_dual_norm: nothing to add")
-    require_cuda(x, y1, y2, bias, gain1, gain2)
+def residual_terms_norm(x: torch.Tensor | None, terms: list[tuple[torch.Tensor, float]], gain1: torch.Tensor | None,
+                        gain2: torch.Tensor | None, eps: float, dtype: torch.dtype, *, bias: torch.Tensor | None = None,
+                        want_stream: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None, torch.Tensor | None]:  # fmt: skip
+    """s = x + sum of f y over the (y, f) of `terms` (at most four) + bias, x and bias optional (float32
+    [n, width]; bias [width]), and its two norms N(s) gain1, N(s) gain2 in `dtype`,
+    N(s) = s / sqrt(mean(s^2) + eps). Returns (s or None, first norm or None, second norm or None)."""
+    first = x if x is not None else (terms[0][0] if terms else None)
+    if first is None or len(terms) > 4:
+        raise KernelLibraryError(f"residual_terms_norm: {len(terms)} terms" if terms else "residual_terms_norm: nothing to add")
+    require_cuda(x, bias, gain1, gain2, *(y for y, _ in terms))
     n, width = first.shape
-    for t, name in ((x, "x"), (y1, "y1"), (y2, "y2")):
-        _rows32(t, name, (n, width))
+    _rows32(x, "x", (n, width))
+    for y, _ in terms:
+        _rows32(y, "a term", (n, width))
     for t, name in ((bias, "bias"), (gain1, "gain1"), (gain2, "gain2")):
         _rows32(t, name, (width,))
     out32 = torch.empty(n, width, device=first.device, dtype=torch.float32) if want_stream else None
     out1 = torch.empty(n, width, device=first.device, dtype=dtype) if gain1 is not None else None
     out2 = torch.empty(n, width, device=first.device, dtype=dtype) if gain2 is not None else None
     code = dtype_code(out1 if out1 is not None else out2) if (out1 is not None or out2 is not None) else 0
-    check(lib().asb_residual_dual_norm(ptr(out32), ptr(out1), ptr(out2), ptr(x), ptr(y1), ptr(y2), ptr(bias), ptr(gain1),
-                                       ptr(gain2), n, width, float(mult), float(eps), code, stream()))  # fmt: skip
+    ys = [ptr(y) for y, _ in terms] + [None] * (4 - len(terms))
+    fs = [float(f) for _, f in terms] + [0.0] * (4 - len(terms))
+    check(lib().asb_residual_terms_norm(ptr(out32), ptr(out1), ptr(out2), ptr(x), *ys, *fs, len(terms), ptr(bias), ptr(gain1),
+                                        ptr(gain2), n, width, float(eps), code, stream()))  # fmt: skip
     return out32, out1, out2
+
+
+def residual_dual_norm(x: torch.Tensor | None, y1: torch.Tensor | None, y2: torch.Tensor | None, mult: float,
+                       gain1: torch.Tensor | None, gain2: torch.Tensor | None, eps: float, dtype: torch.dtype, *,
+                       bias: torch.Tensor | None = None,
+                       want_stream: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None, torch.Tensor | None]:  # fmt: skip
+    """`residual_terms_norm` of x + mult (y1 + y2) + bias, every term optional."""
+    terms = [(y, mult) for y in (y1, y2) if y is not None]
+    return residual_terms_norm(x, terms, gain1, gain2, eps, dtype, bias=bias, want_stream=want_stream)
 
 
 def pair_embedding(ids: torch.Tensor, positions: torch.Tensor, req_q_start: torch.Tensor, state_slots: torch.Tensor,

@@ -4,6 +4,10 @@ and no biases. Sizes, eps, the position encoding, the score scale and the window
 `names` gives the checkpoint's tensor names where they are not the `*_proj.weight` ones, and
 `value_dim` a value size that differs from the key size.
 
+`norm_over="projection"`: q and k are RMS-normed over all their heads at once (gains of the whole
+projection's size) instead of head by head. `fixed_sink`: every head's softmax has one more term
+exp(fixed_sink) in its denominator, with no key, no value and no learned logit.
+
 Where value_dim != head_dim the pages and kernels run at the larger of the two: the narrower of
 (queries and keys) and (values) is padded with zero rows in the loaded weights, which changes no
 score and no output (the q/k norm's mean is taken over head_dim entries: the gains carry
@@ -36,6 +40,8 @@ class GQAttention(Mixer):
         softcap: float | None = None,
         query_temperature: tuple[float, int] | None = None,
         chunk: int | None = None,
+        norm_over: str = "head",
+        fixed_sink: float | None = None,
     ):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads are not a multiple of {num_kv_heads} kv heads")
@@ -59,6 +65,11 @@ class GQAttention(Mixer):
         self.query_temperature = (float(query_temperature[0]), int(query_temperature[1])) if query_temperature else None
         if self.query_temperature is not None and (qk_norm_eps is not None or self.query_temperature[1] < 1):
             raise ValueError("a query temperature goes with unnormed queries and a positive period")
+        if norm_over not in ("head", "projection") or (norm_over == "projection" and (qk_norm_eps is None or self.query_temperature is not None)):
+            raise ValueError(f"norm_over {norm_over!r}: 'head', or 'projection' for normed queries without a temperature")
+        if fixed_sink is not None and sink:
+            raise ValueError("a sink is learned or fixed, not both")
+        self.norm_over, self.fixed_sink = norm_over, fixed_sink
         self.qkv_proj = self.o_proj = self.q_gain = self.k_gain = self.sink = None
 
     def cache_spec(self) -> PageSpec:
@@ -73,9 +84,10 @@ class GQAttention(Mixer):
             TensorSpec(n["o"], (d, self.num_heads * vd)),
         ]
         if self.qk_norm_eps is not None:
+            whole = self.norm_over == "projection"
             specs += [
-                TensorSpec(n["q_norm"], (kd,), kind="gain", init="gain"),
-                TensorSpec(n["k_norm"], (kd,), kind="gain", init="gain"),
+                TensorSpec(n["q_norm"], (self.num_heads * kd if whole else kd,), kind="gain", init="gain"),
+                TensorSpec(n["k_norm"], (self.num_kv_heads * kd if whole else kd,), kind="gain", init="gain"),
             ]
         if self.has_sink:
             specs.append(TensorSpec(n["sink"], (self.num_heads,), kind="gain", init="normal"))
@@ -84,8 +96,10 @@ class GQAttention(Mixer):
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         n, hd, kd, vd = self.names, self.head_dim, self.key_dim, self.value_dim
 
+        whole = self.norm_over == "projection"  # (whose kernel pads heads itself: the stack stays as it is)
+
         def rows_per_head(w: torch.Tensor, heads: int, size: int) -> torch.Tensor:
-            if size == hd:
+            if size == hd or whole:
                 return w
             padded = w.new_zeros(heads, hd, w.shape[1])
             padded[:, :size] = w.view(heads, size, w.shape[1])
@@ -102,10 +116,12 @@ class GQAttention(Mixer):
             o[:, :, :vd] = self.o_proj.view(-1, self.num_heads, vd)
             self.o_proj = o.view(-1, self.num_heads * hd).contiguous()
         self.sink = tensors[n["sink"]].contiguous() if self.has_sink else None
+        if self.fixed_sink is not None:
+            self.sink = torch.full((self.num_heads,), float(self.fixed_sink), dtype=torch.float32, device=self.o_proj.device)
         self.kernel_eps = self.qk_norm_eps
         if self.qk_norm_eps is not None:
             self.q_gain, self.k_gain = tensors[n["q_norm"]], tensors[n["k_norm"]]
-            if kd != hd:
+            if kd != hd and not whole:
                 pad = (kd / hd) ** 0.5
                 self.q_gain = torch.cat([self.q_gain * pad, self.q_gain.new_zeros(hd - kd)]).contiguous()
                 self.k_gain = torch.cat([self.k_gain * pad, self.k_gain.new_zeros(hd - kd)]).contiguous()
@@ -113,11 +129,13 @@ class GQAttention(Mixer):
         if self.position is not None:
             self.position.prepare(self.o_proj.device)
             rotary = self.position.fused_rotary()
+            if rotary is None and whole:
+                raise NotImplementedError("queries normed over the whole projection take positions as a fused rotation")
             if rotary is not None and rotary.magnitude != 1.0:
                 # cosines and sines times a constant: the turned entries of q and k times it, which
                 # the gains of the norm before the rotation carry (a pair's two entries both turn)
-                if self.qk_norm_eps is None:
-                    raise NotImplementedError("a rotation with a magnitude needs the q/k norm, whose gains carry it")
+                if self.qk_norm_eps is None or whole:
+                    raise NotImplementedError("a rotation with a magnitude needs the per-head q/k norm, whose gains carry it")
                 scale = torch.ones_like(self.q_gain)
                 scale[: rotary.rotary_dim] = rotary.magnitude
                 self.q_gain, self.k_gain = (self.q_gain * scale).contiguous(), (self.k_gain * scale).contiguous()
@@ -140,9 +158,35 @@ class GQAttention(Mixer):
         projection's partial sums for the norm that follows to add up (`ops.linear_for_stream`)."""
         return ops.linear_for_stream(self.attend(h, ctx, cache, write_cache), self.o_proj)
 
+    def input_weights(self) -> torch.Tensor:
+        """The stacked input projection, for a mixer that runs this one beside another and
+        multiplies once for both (`forward_from` then reads this one's columns of the product)."""
+        if self.norm_over != "projection":
+            raise NotImplementedError("attention beside another mixer norms its queries over the whole projection")
+        return self.qkv_proj
+
+    def forward_from(self, proj: torch.Tensor, col: int, ctx: StepContext, cache: CacheView, write_cache: bool = True) -> torch.Tensor:
+        return ops.linear(self.attend_from(proj, col, ctx, cache, write_cache), self.o_proj, out_dtype=torch.float32)
+
+    def attend_from(self, proj: torch.Tensor, col: int, ctx: StepContext, cache: CacheView, write_cache: bool) -> torch.Tensor:
+        """`attend` for queries and keys normed over the whole projection, from a product that holds this
+        mixer's projection in the columns from `col`."""
+        H, KV, hd = self.num_heads, self.num_kv_heads, self.head_dim
+        rotary = self.position.fused_rotary() if self.position is not None else None
+        q = ops.projection_norm_rope_store(
+            proj, col, H, KV, self.key_dim, self.value_dim, hd, ctx.positions, self.q_gain, self.k_gain, self.qk_norm_eps,
+            inv_freq=rotary.inv_freq if rotary else None, rotary_dim=rotary.rotary_dim if rotary else 0,
+            interleaved=rotary is not None and rotary.pairing == "interleaved", slots=cache.slots if write_cache else None,
+            k_cache=cache.k if write_cache else None, v_cache=cache.v if write_cache else None,
+        )  # fmt: skip
+        return self._over_pages(q, ctx, cache)
+
     def attend(self, h: torch.Tensor, ctx: StepContext, cache: CacheView | None, write_cache: bool) -> torch.Tensor:
         """The heads' outputs side by side, [T, H * hd], before the output projection."""
         H, KV, hd = self.num_heads, self.num_kv_heads, self.head_dim
+        if self.norm_over == "projection":
+            weight = self.qkv_proj if write_cache else self.qkv_proj[: H * self.key_dim]
+            return self.attend_from(ops.linear(h, weight), 0, ctx, cache, write_cache)
         # the position encoding says how it is applied: by the fused kernel below (a rotation by
         # position x frequency), or by its own `encode` on the normalised queries and keys
         rotary = self.position.fused_rotary() if self.position is not None else None
@@ -176,13 +220,15 @@ class GQAttention(Mixer):
                 slots=cache.slots if write_cache else None,
                 k_cache=cache.k if write_cache else None, v_cache=cache.v if write_cache else None,
             )  # fmt: skip
+        return self._over_pages(q, ctx, cache)
+
+    def _over_pages(self, q: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
         out = ops.paged_attention(
             q, cache.k, cache.v, cache.block_tables, ctx.req_q_start, ctx.req_pos_start,
             num_requests=ctx.num_requests, max_context=ctx.max_context, window=self.window,
             scale=self.scale, host_q_lens=ctx.host_q_lens or None, sink=self.sink, chunk=self.chunk, softcap=self.softcap,
         )  # fmt: skip
-        return out.view(-1, H * hd)
-
+        return out.view(-1, self.num_heads * self.head_dim)
 
     def _project_encode_store(self, h: torch.Tensor, ctx: StepContext, cache: CacheView | None, write_cache: bool) -> torch.Tensor:
         """The path for an encoding that is no fused rotation: the same kernel normalises q and k

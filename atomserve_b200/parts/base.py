@@ -329,6 +329,6 @@ def build_block(kind: str, mixer: Mixer, feed_forward: FeedForward, mixer_norm: 
 def _ensure_builtin() -> None:
     if "rms_norm" not in _REGISTRIES["norm"]:
         from atomserve_b200.parts import (  # noqa: F401
-            attention, block, differential_attention, embedding, experts, latent_attention, lightning, matrix_memory, mixed_heads, mlp,
+            attention, block, delta_rule, differential_attention, embedding, experts, latent_attention, lightning, matrix_memory, mixed_heads, mlp,
             norms, parallel, rotary, sink_attention, state_space, stream_step, token_input,
         )

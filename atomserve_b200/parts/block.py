@@ -148,7 +148,8 @@ class ParallelResidualBlock(PostNormBlock):
     """The arrangement in which mixer and feed-forward read the same float32 stream, each through
     an RMS norm of its own, and are added together: x <- x + mult (mixer(N1 x) + ff(N2 x)); a layer
     without a feed-forward adds the mixer alone. The norms are `RMSNorm`s; `mult` is the mixer
-    norm's `mult` (`ScaledRMSNorm`), 1 without one. The kernel that adds a layer's two outputs also
+    norm's `mult` (`ScaledRMSNorm`), 1 without one. A mixer that offers `forward_terms` gives its output
+    as several float32 terms with a factor each. The kernel that adds a layer's outputs also
     norms the sum twice for the next block of this kind, so the pair (N1 x, N2 x) travels from
     block to block in the place where pre-norm blocks hand on their normed input. Sublayers give
     float32 outputs (`forward_for_stream` must not leave partial sums: two products are added)."""
@@ -167,13 +168,16 @@ class ParallelResidualBlock(PostNormBlock):
             _, h1, h2 = ops.residual_dual_norm(x, None, None, 1.0, g1, g2, eps, self.dtype, want_stream=False)
         else:
             h1, h2 = normed
-        y1 = self.mixer.forward(h1, None, ctx, cache, write_cache)
-        y2 = self.feed_forward.forward(h2, None, ctx) if self.has_feed_forward else None
+        several = getattr(self.mixer, "forward_terms", None)
+        terms = several(h1, ctx, cache, write_cache) if several is not None else [(self.mixer.forward(h1, None, ctx, cache, write_cache), 1.0)]
+        if self.has_feed_forward:
+            terms.append((self.feed_forward.forward(h2, None, ctx), 1.0))
+        terms = [(y, f * self.mult) for y, f in terms]
         owner = getattr(then, "block_norms", None) if then is not None else None
         if owner is None:  # the last block, or one of another kind next: the sum alone
-            return ops.residual_dual_norm(x, y1, y2, self.mult, None, None, 0.0, self.dtype)[0], None
+            return ops.residual_terms_norm(x, terms, None, None, 0.0, self.dtype)[0], None
         n1, n2, eps_next = owner()
-        x, h1, h2 = ops.residual_dual_norm(x, y1, y2, self.mult, n1, n2, eps_next, self.dtype)
+        x, h1, h2 = ops.residual_terms_norm(x, terms, n1, n2, eps_next, self.dtype)
         return x, (h1, h2)
 
     def bind_dtype(self, dtype: torch.dtype) -> None:

@@ -11,17 +11,21 @@ from atomserve_b200.parts.spec import TensorSpec
 
 
 class RMSNorm(Norm):
-    def __init__(self, hidden_size: int, prefix: str, eps: float, width: int | None = None, tensor: str | None = None):
+    """`centre`: what the gain is stored less of (1 for a checkpoint that keeps gains around zero); the
+    gain the kernels read is made once at load, in float32."""
+
+    def __init__(self, hidden_size: int, prefix: str, eps: float, width: int | None = None, tensor: str | None = None,
+                 centre: float = 0.0):  # fmt: skip
         self.width = width or hidden_size
-        self.eps = float(eps)
+        self.eps, self.centre = float(eps), float(centre)
         self.name = tensor or prefix + "weight"
         self.gain: torch.Tensor | None = None
 
     def tensor_specs(self) -> list[TensorSpec]:
-        return [TensorSpec(self.name, (self.width,), kind="gain", init="gain")]
+        return [TensorSpec(self.name, (self.width,), kind="gain", init="normal" if self.centre else "gain")]
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
-        self.gain = tensors[self.name]
+        self.gain = tensors[self.name] + self.centre if self.centre else tensors[self.name]
 
     def forward(self, x: torch.Tensor, rows: torch.Tensor | None = None) -> torch.Tensor:
         return ops.rms_norm(x, self.gain, self.eps, rows)
@@ -44,8 +48,8 @@ class ScaledRMSNorm(RMSNorm):
     sublayers give before adding it to the stream (blocks that sum their sublayers themselves)."""
 
     def __init__(self, hidden_size: int, prefix: str, eps: float, mult: float = 1.0, width: int | None = None,
-                 tensor: str | None = None):  # fmt: skip
-        super().__init__(hidden_size, prefix, eps, width, tensor)
+                 tensor: str | None = None, centre: float = 0.0):  # fmt: skip
+        super().__init__(hidden_size, prefix, eps, width, tensor, centre)
         self.mult = float(mult)
 
 
@@ -56,8 +60,8 @@ class StreamRMSNorm(RMSNorm):
     the plain norm of (rows of) the stream in the compute dtype, as a final norm before the head."""
 
     def __init__(self, hidden_size: int, prefix: str, eps: float, alpha: float = 1.0, width: int | None = None,
-                 tensor: str | None = None):  # fmt: skip
-        super().__init__(hidden_size, prefix, eps, width, tensor)
+                 tensor: str | None = None, centre: float = 0.0):  # fmt: skip
+        super().__init__(hidden_size, prefix, eps, width, tensor, centre)
         self.alpha = float(alpha)
         self.dtype = torch.float32
 

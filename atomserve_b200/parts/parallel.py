@@ -1,8 +1,10 @@
-"""Two mixers side by side as one: both read the same input, and the result is half the sum of
-their outputs, each RMS-normed over the model width with a gain of its own,
-(R(left(h)) gain_left + R(right(h)) gain_right) / 2. The two are given as part descriptions; what
-either keeps between steps (pages, state) is this mixer's: at most one of them may keep pages.
-Their input projections are stacked, so the input is multiplied once for both."""
+"""Two mixers side by side as one: both read the same input. The two are given as part descriptions;
+what either keeps between steps (pages, state) is this mixer's: at most one of them may keep pages.
+Their input projections are stacked, so the input is multiplied once for both.
+
+`ParallelMixers`: half the sum of their outputs, each RMS-normed over the model width with a gain of
+its own, (R(left(h)) gain_left + R(right(h)) gain_right) / 2.
+`WeightedMixers`: left_scale left(h) + right_scale right(h)."""
 
 from __future__ import annotations
 
@@ -13,12 +15,12 @@ from atomserve_b200.parts.base import CacheView, Mixer, PageSpec, StateSpec, Ste
 from atomserve_b200.parts.spec import PartSpec, TensorSpec
 
 
-class ParallelMixers(Mixer):
-    def __init__(self, hidden_size: int, prefix: str, left: PartSpec, right: PartSpec, eps: float,
-                 left_gain: str | None = None, right_gain: str | None = None):  # fmt: skip
-        self.hidden_size, self.eps = hidden_size, float(eps)
+class MixerPair(Mixer):
+    """What the two kinds of pairs share: the two parts, what they keep, and their stacked projection."""
+
+    def __init__(self, hidden_size: int, left: PartSpec, right: PartSpec):
+        self.hidden_size = hidden_size
         self.left, self.right = build_part("mixer", left, hidden_size), build_part("mixer", right, hidden_size)
-        self.names = (left_gain or prefix + "left.out", right_gain or prefix + "right.out")
         for side in (self.left, self.right):
             if not hasattr(side, "input_weights") or not hasattr(side, "forward_from"):
                 raise ValueError(f"{type(side).__name__} cannot run beside another mixer (no input_weights / forward_from)")
@@ -27,7 +29,7 @@ class ParallelMixers(Mixer):
         names = [s.name for side in (self.left, self.right) for s in side.state_specs()]
         if len(set(names)) != len(names):
             raise ValueError(f"the two mixers' state names collide: {names}")
-        self.in_proj = self.gains = None
+        self.in_proj = None
         self.split = 0
 
     @property
@@ -41,8 +43,7 @@ class ParallelMixers(Mixer):
         return self.left.state_specs() + self.right.state_specs()
 
     def tensor_specs(self) -> list[TensorSpec]:
-        own = [TensorSpec(n, (self.hidden_size,), kind="gain", init="gain") for n in self.names]
-        return self.left.tensor_specs() + self.right.tensor_specs() + own
+        return self.left.tensor_specs() + self.right.tensor_specs()
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         self.left.load(tensors)
@@ -50,14 +51,40 @@ class ParallelMixers(Mixer):
         a, b = self.left.input_weights(), self.right.input_weights()
         self.split = a.shape[0]
         self.in_proj = torch.cat([a, b]).contiguous()
+
+    def outputs(self, h: torch.Tensor, ctx: StepContext, cache: CacheView | None, write_cache: bool) -> tuple[torch.Tensor, torch.Tensor]:
+        """(left(h), right(h)), float32."""
+        proj = ops.linear(h, self.in_proj)
+
+        def run(side: Mixer, col: int) -> torch.Tensor:
+            more = {}
+            if side.cache_spec() is not None:
+                more["write_cache"] = write_cache
+            if getattr(side, "reads_input", False):  # a side with projections outside the stack
+                more["h"] = h
+            return side.forward_from(proj, col, ctx, cache, **more)
+
+        return run(self.left, 0), run(self.right, self.split)
+
+
+class ParallelMixers(MixerPair):
+    def __init__(self, hidden_size: int, prefix: str, left: PartSpec, right: PartSpec, eps: float,
+                 left_gain: str | None = None, right_gain: str | None = None):  # fmt: skip
+        super().__init__(hidden_size, left, right)
+        self.eps, self.gains = float(eps), None
+        self.names = (left_gain or prefix + "left.out", right_gain or prefix + "right.out")
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        own = [TensorSpec(n, (self.hidden_size,), kind="gain", init="gain") for n in self.names]
+        return super().tensor_specs() + own
+
+    def load(self, tensors: dict[str, torch.Tensor]) -> None:
+        super().load(tensors)
         self.gains = tuple(tensors[n] for n in self.names)
 
     def forward_halves(self, h: torch.Tensor, ctx: StepContext, cache: CacheView | None, write_cache: bool = True):
         """(left(h), (right(h), gain_left, gain_right)), float32: for a block whose norm kernel joins them."""
-        proj = ops.linear(h, self.in_proj)
-        takes_write = lambda side: side.cache_spec() is not None  # noqa: E731
-        a = self.left.forward_from(proj, 0, ctx, cache, write_cache) if takes_write(self.left) else self.left.forward_from(proj, 0, ctx, cache)
-        b = self.right.forward_from(proj, self.split, ctx, cache, write_cache) if takes_write(self.right) else self.right.forward_from(proj, self.split, ctx, cache)
+        a, b = self.outputs(h, ctx, cache, write_cache)
         return a, (b, *self.gains)
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor | None, ctx: StepContext,
@@ -77,4 +104,21 @@ def _join(a: torch.Tensor, b: torch.Tensor, ga: torch.Tensor, gb: torch.Tensor, 
     return (na + nb) * 0.5
 
 
+class WeightedMixers(MixerPair):
+    def __init__(self, hidden_size: int, prefix: str, left: PartSpec, right: PartSpec, left_scale: float, right_scale: float):
+        super().__init__(hidden_size, left, right)
+        self.scales = (float(left_scale), float(right_scale))
+
+    def forward_terms(self, h: torch.Tensor, ctx: StepContext, cache: CacheView | None, write_cache: bool = True):
+        """The two outputs with their factors, float32: for a block whose sum takes several terms."""
+        return list(zip(self.outputs(h, ctx, cache, write_cache), self.scales))
+
+    def forward(self, h: torch.Tensor, residual: torch.Tensor | None, ctx: StepContext,
+                cache: CacheView | None, write_cache: bool = True) -> torch.Tensor:  # fmt: skip
+        # (blocks that sum their sublayers in float32 themselves take `forward_terms`)
+        joined = ops.residual_terms_norm(None, self.forward_terms(h, ctx, cache, write_cache), None, None, 0.0, torch.float32)[0]
+        return joined if residual is None else residual + joined.to(residual.dtype)
+
+
 register_part("mixer", "parallel_mixers", ParallelMixers)
+register_part("mixer", "weighted_mixers", WeightedMixers)

@@ -51,4 +51,23 @@ class MixWithInput(StreamStep):
         return x, (h1, h2)
 
 
+class AddInput(StreamStep):
+    def __init__(self, hidden_size: int, prefix: str):
+        self.dtype = torch.float32
+
+    def bind_dtype(self, dtype: torch.dtype) -> None:
+        self.dtype = dtype
+
+    def forward(self, x: torch.Tensor, x0: torch.Tensor, number: int, ctx: StepContext) -> torch.Tensor:
+        return self.forward_then(x, x0, number, ctx, None)[0]
+
+    def forward_then(self, x: torch.Tensor, x0: torch.Tensor, number: int, ctx: StepContext, then):
+        """As `MixWithInput.forward_then`."""
+        owner = getattr(then, "block_norms", None) if then is not None else None
+        g1, g2, eps = owner() if owner is not None else (None, None, 0.0)
+        x, h1, h2 = ops.residual_terms_norm(x, [(x0, 1.0)], g1, g2, eps, self.dtype)
+        return x, ((h1, h2) if owner is not None else None)
+
+
+register_part("stream_step", "add_input", AddInput)
 register_part("stream_step", "mix_with_input", MixWithInput)
