@@ -22,8 +22,6 @@ what such rounding alone does to the logits.
 
 from __future__ import annotations
 
-import math
-
 import torch
 
 F64 = torch.float64
@@ -56,12 +54,12 @@ def turn_halves(x: torch.Tensor, base: float, dims: int, first: int = 0) -> torc
     i + dims / 2, the pair turned by position * base^(-2 i / dims); the rest passes."""
     half = dims // 2
     out = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(half):
-            a = (first + t) * base ** (-2.0 * i / dims)
-            u, v = x[t, :, i], x[t, :, i + half]
-            out[t, :, i] = u * math.cos(a) - v * math.sin(a)
-            out[t, :, i + half] = v * math.cos(a) + u * math.sin(a)
+    p = torch.arange(first, first + x.shape[0], dtype=F64)[:, None]
+    for i in range(half):
+        a = p * base ** (-2.0 * i / dims)
+        u, v = x[:, :, i], x[:, :, i + half]
+        out[:, :, i] = u * torch.cos(a) - v * torch.sin(a)
+        out[:, :, i + half] = v * torch.cos(a) + u * torch.sin(a)
     return out
 
 
