@@ -292,11 +292,40 @@ delta_chunk_prepare_kernel(const ChunkParams p) {
   const int row0 = p.chunk_row[chunk], n = p.chunk_len[chunk];
   const size_t at = (size_t)chunk * in.H + h;
   // rows past the chunk's tokens: zero vectors, beta 0, decay 1; they change nothing
-  for (int i = warp; i < C; i += kPrepareThreads / 32) {
-    if (i < n) {
-      unit_qk<T>(in, (size_t)(row0 + i), h, qs + i * LD, ks + i * LD, DP, lane);
-    } else {
-      for (int d = lane; d < DP; d += 32) qs[i * LD + d] = ks[i * LD + d] = 0.f;
+  // (four rows a warp at a time, their loads in flight together)
+  for (int i0 = warp * 4; i0 < C; i0 += kPrepareThreads / 8) {
+    const T* src = (const T*)in.x + (size_t)(row0 + i0) * in.stride + (h / in.share) * in.D;
+    float qq[4] = {0.f, 0.f, 0.f, 0.f}, kk[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int d = lane; d < DP; d += 32) {
+      float q[4], k[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const bool real = i0 + u < n && d < in.D;
+        q[u] = real ? asb::to_float(src[(size_t)u * in.stride + in.q_off + d]) : 0.f;
+        k[u] = real ? asb::to_float(src[(size_t)u * in.stride + in.k_off + d]) : 0.f;
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        qs[(i0 + u) * LD + d] = q[u];
+        ks[(i0 + u) * LD + d] = k[u];
+        qq[u] = fmaf(q[u], q[u], qq[u]);
+        kk[u] = fmaf(k[u], k[u], kk[u]);
+      }
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        qq[u] += __shfl_xor_sync(0xffffffffu, qq[u], off);
+        kk[u] += __shfl_xor_sync(0xffffffffu, kk[u], off);
+      }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const float rq = in.q_scale / sqrtf(qq[u] + kUnitEps), rk = 1.f / sqrtf(kk[u] + kUnitEps);
+      for (int d = lane; d < DP; d += 32) {  // (each lane rescales what it wrote)
+        qs[(i0 + u) * LD + d] *= rq;
+        ks[(i0 + u) * LD + d] *= rk;
+      }
     }
   }
   if (warp == 0) {
@@ -334,7 +363,7 @@ delta_chunk_prepare_kernel(const ChunkParams p) {
         const float4 kr = *reinterpret_cast<const float4*>(ks + (ti + 16 * a) * LD + d);
         const float4 qr = *reinterpret_cast<const float4*>(qs + (ti + 16 * a) * LD + d);
 #pragma unroll
-        for (int b = 0; b < TI; ++b) {
+        for (int b = 0; b <= a; ++b) {  // (sub-blocks above the diagonal are not needed)
           kk[a][b] = fmaf(kr.x, kc[b].x, fmaf(kr.y, kc[b].y, fmaf(kr.z, kc[b].z, fmaf(kr.w, kc[b].w, kk[a][b]))));
           qk[a][b] = fmaf(qr.x, kc[b].x, fmaf(qr.y, kc[b].y, fmaf(qr.z, kc[b].z, fmaf(qr.w, kc[b].w, qk[a][b]))));
         }
@@ -346,6 +375,11 @@ delta_chunk_prepare_kernel(const ChunkParams p) {
 #pragma unroll
       for (int b = 0; b < TI; ++b) {
         const int i = ti + 16 * a, j = tj + 16 * b;
+        if (b > a) {
+          L[i * LA + j] = 0.f;
+          pt[j * C + i] = 0.f;
+          continue;
+        }
         const float e = j <= i ? expf(G[i] - G[j]) : 0.f;  // (above the diagonal the exponent may be large)
         L[i * LA + j] = j < i ? beta[i] * e * kk[a][b] : 0.f;
         pt[j * C + i] = e * qk[a][b];
@@ -354,16 +388,15 @@ delta_chunk_prepare_kernel(const ChunkParams p) {
   // e^(G_C - G) K, and e^G Q as columns
   const float last = G[C - 1];
   float* kd = p.kd + at * C * DP;
-  for (int idx = tid; idx < C * DP; idx += kPrepareThreads) {
-    const int i = idx / DP, d = idx - i * DP;
-    kd[idx] = ks[i * LD + d] * expf(last - G[i]);
+  for (int i = warp; i < C; i += kPrepareThreads / 32) {
+    const float e = expf(last - G[i]);
+    for (int d = lane; d < DP; d += 32) kd[i * DP + d] = ks[i * LD + d] * e;
   }
   float* wq = p.wq + at * DP * 2 * C;
-  for (int idx = tid; idx < DP * (C / 4); idx += kPrepareThreads) {
-    const int i = idx / DP * 4, d = idx % DP;
-    *reinterpret_cast<float4*>(wq + (size_t)d * 2 * C + C + i) =
-        make_float4(qs[i * LD + d] * eg[i], qs[(i + 1) * LD + d] * eg[i + 1], qs[(i + 2) * LD + d] * eg[i + 2], qs[(i + 3) * LD + d] * eg[i + 3]);
-  }
+  for (int i = warp * 4; i < C; i += kPrepareThreads / 8)
+    for (int d = lane; d < DP; d += 32)
+      *reinterpret_cast<float4*>(wq + (size_t)d * 2 * C + C + i) =
+          make_float4(qs[i * LD + d] * eg[i], qs[(i + 1) * LD + d] * eg[i + 1], qs[(i + 2) * LD + d] * eg[i + 2], qs[(i + 3) * LD + d] * eg[i + 3]);
   if (tid == 0) p.through[at] = eg[C - 1];
   __syncthreads();
   // (I + L) X = diag(beta) [V | e^G K], a column a thread, forward substitution in registers
@@ -404,16 +437,37 @@ delta_chunk_prepare_kernel(const ChunkParams p) {
   }
 }
 
-template <int N>
+// acc += A B over k_end (a multiple of 4) values of k, A's rows and B's columns four at a time from shared
+// memory, the next four k's operands on their way while these are multiplied
 __device__ __forceinline__ void multiply_add(float (&acc)[4][4], const float* a, int a_stride, const float* b, int b_stride, int k_end) {
-#pragma unroll N
-  for (int k = 0; k < k_end; ++k) {
-    const float4 av = *reinterpret_cast<const float4*>(a + k * a_stride), bv = *reinterpret_cast<const float4*>(b + k * b_stride);
-    const float x[4] = {av.x, av.y, av.z, av.w}, w[4] = {bv.x, bv.y, bv.z, bv.w};
+  float4 av[4], bv[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+  for (int u = 0; u < 4; ++u) {
+    av[u] = *reinterpret_cast<const float4*>(a + u * a_stride);
+    bv[u] = *reinterpret_cast<const float4*>(b + u * b_stride);
+  }
+#pragma unroll 2
+  for (int k = 0; k < k_end; k += 4) {
+    float4 an[4], bn[4];
+    const int next = k + 4 < k_end ? k + 4 : 0;  // (past the end: any operands, never used)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], w[j], acc[i][j]);
+    for (int u = 0; u < 4; ++u) {
+      an[u] = *reinterpret_cast<const float4*>(a + (next + u) * a_stride);
+      bn[u] = *reinterpret_cast<const float4*>(b + (next + u) * b_stride);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const float x[4] = {av[u].x, av[u].y, av[u].z, av[u].w}, w[4] = {bv[u].x, bv[u].y, bv[u].z, bv[u].w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], w[j], acc[i][j]);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      av[u] = an[u];
+      bv[u] = bn[u];
+    }
   }
 }
 
@@ -423,16 +477,17 @@ __device__ __forceinline__ void fetch(float* dst, const float* src, int count) {
   for (int i = threadIdx.x * 4; i < count; i += THREADS * 4) cp_async16(smem_u32(dst + i), src + i, true);
 }
 
+// Two groups of threads, each with a thread per 4 x 4 tile of [W ; Q] S.
 template <int C, int VS>
 struct Walk {
-  static constexpr int kThreads = (2 * C / 4) * (VS / 4);
-  static constexpr size_t floats(int DP) { return (size_t)DP * 2 * C + (size_t)C * DP + C * C + 2 * C * VS + (size_t)DP * VS; }
+  static constexpr int kGroup = (2 * C / 4) * (VS / 4), kThreads = 2 * kGroup;
+  static constexpr size_t floats(int DP) { return (size_t)DP * 2 * C + (size_t)C * DP + C * C + 4 * C * VS + (size_t)DP * VS; }
 };
 
 template <int C, int VS>
 __global__ void __launch_bounds__(Walk<C, VS>::kThreads)
 delta_chunk_walk_kernel(const ChunkParams p) {
-  constexpr int NT = Walk<C, VS>::kThreads, CT = VS / 4;
+  constexpr int NG = Walk<C, VS>::kGroup, NT = Walk<C, VS>::kThreads, CT = VS / 4;
   extern __shared__ __align__(16) float smem[];
   const DeltaInputs& in = p.in;
   const int DP = p.DP, V = in.V, H = in.H;
@@ -442,6 +497,7 @@ delta_chunk_walk_kernel(const ChunkParams p) {
   float* y = pt + C * C;            // [C][VS]
   float* u = y + C * VS;            // [C][VS]
   float* S = u + C * VS;            // [DP][VS]
+  float* second = S + DP * VS;      // [2 C][VS]: the second group's share of [W ; Q] S
   asb::pdl_wait();
   asb::pdl_launch_dependents();
   const int tid = threadIdx.x, h = blockIdx.y, v0 = blockIdx.z * VS;
@@ -466,8 +522,11 @@ delta_chunk_walk_kernel(const ChunkParams p) {
     const int d = i / VS, c = i - d * VS;
     S[i] = (d < in.D && v0 + c < V) ? sp[(size_t)d * V + c] : 0.f;
   }
-  const int rt = tid / CT, ct = tid % CT;     // a thread's tile: 4 rows of [W ; Q] by 4 columns
-  const bool solves = rt < C / 4;             // this half makes U and the new S, the other half O
+  // [W ; Q] S: both groups, each over its half of the rows of S; then the first group makes U (its tiles of W)
+  // and O (those of Q) and the second the new S
+  const bool first = tid < NG;
+  const int t = first ? tid : tid - NG, rt = t / CT, ct = t % CT;
+  const int k_half = (DP / 4 + 1) / 2 * 4, k_from = first ? 0 : k_half, k_count = first ? k_half : DP - k_half;
   for (int c = c_first; c < c_end; ++c) {
     const int row0 = p.chunk_row[c], n = p.chunk_len[c];
     const float through = p.through[(size_t)c * H + h];
@@ -478,23 +537,45 @@ delta_chunk_walk_kernel(const ChunkParams p) {
     for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    multiply_add<8>(acc, wq + rt * 4, 2 * C, S + ct * 4, VS, DP);
-    if (solves) {
+    if (k_count > 0) multiply_add(acc, wq + k_from * 2 * C + rt * 4, 2 * C, S + k_from * VS + ct * 4, VS, k_count);
+    if (!first) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(second + (rt * 4 + i) * VS + ct * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    }
+    __syncthreads();  // W and Q have been read
+    if (first) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int at = (rt * 4 + i) * VS + ct * 4;
-        const float4 own = *reinterpret_cast<const float4*>(y + at);
-        *reinterpret_cast<float4*>(u + at) = make_float4(own.x - acc[i][0], own.y - acc[i][1], own.z - acc[i][2], own.w - acc[i][3]);
+        const float4 rest = *reinterpret_cast<const float4*>(second + at);
+        acc[i][0] += rest.x; acc[i][1] += rest.y; acc[i][2] += rest.z; acc[i][3] += rest.w;
+        if (rt < C / 4) {
+          const float4 own = *reinterpret_cast<const float4*>(y + at);
+          *reinterpret_cast<float4*>(u + at) = make_float4(own.x - acc[i][0], own.y - acc[i][1], own.z - acc[i][2], own.w - acc[i][3]);
+        }
       }
     }
-    __syncthreads();  // U is there, and W, Q and Y have been read
+    cp_async_wait<0>();  // (K and P of this chunk)
+    __syncthreads();     // U is there, and Y has been read
     if (c + 1 < c_end) fetch_first(c + 1);
     cp_async_commit();
-    cp_async_wait<1>();
-    __syncthreads();  // K and P of this chunk are there
-    if (!solves) {
+    if (!first) {
+      for (int tile = t; tile < DP / 4 * CT; tile += NG) {
+        const int d0 = tile / CT * 4, c0 = tile % CT * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 s = *reinterpret_cast<const float4*>(S + (d0 + i) * VS + c0);
+          acc[i][0] = through * s.x; acc[i][1] = through * s.y; acc[i][2] = through * s.z; acc[i][3] = through * s.w;
+        }
+        multiply_add(acc, kd + d0, DP, u + c0, VS, C);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          *reinterpret_cast<float4*>(S + (d0 + i) * VS + c0) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+      }
+    } else if (rt >= C / 4) {
       const int i0 = rt * 4 - C;
-      multiply_add<8>(acc, pt + i0, C, u + ct * 4, VS, C);
+      multiply_add(acc, pt + i0, C, u + ct * 4, VS, C);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         if (i0 + i >= n) break;
@@ -506,19 +587,6 @@ delta_chunk_walk_kernel(const ChunkParams p) {
           for (int j = 0; j < 4; ++j)
             if (v0 + ct * 4 + j < V) o[j] = acc[i][j];
         }
-      }
-    } else {
-      for (int tile = tid; tile < DP / 4 * CT; tile += NT / 2) {
-        const int d0 = tile / CT * 4, c0 = tile % CT * 4;
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float4 s = *reinterpret_cast<const float4*>(S + (d0 + i) * VS + c0);
-          acc[i][0] = through * s.x; acc[i][1] = through * s.y; acc[i][2] = through * s.z; acc[i][3] = through * s.w;
-        }
-        multiply_add<8>(acc, kd + d0, DP, u + c0, VS, C);
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          *reinterpret_cast<float4*>(S + (d0 + i) * VS + c0) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
       }
     }
     __syncthreads();  // S is new, and K, P and U have been read

@@ -6,6 +6,9 @@
 //                            written as the float32 stream, and N(s) gain1, N(s) gain2 in the compute
 //                            dtype, N(s) = s / sqrt(mean(s^2) + eps): the sum of a layer, whatever
 //                            number of outputs it has, and both norms of the next one in one pass
+//   asb_partial_residual_terms_norm  the same with one more term given as the partial sums that the
+//                            tensor-core GEMM left in its workspace (few tokens): a thread adds up the
+//                            slots of 8 columns itself, in the order of the GEMM's own reduction
 //   asb_pair_embedding       x[t] = table[id[t]] + pairs[row(previous id, id[t])], float32: a
 //                            hashed table of token pairs beside the token table. The id before a
 //                            request's first token of the step is per-request state (0: none yet)
@@ -14,6 +17,7 @@
 //
 // Sums and norms are float32; each stored value is rounded once.
 #include "common.cuh"
+#include "gemm_partials.cuh"
 
 namespace {
 
@@ -124,6 +128,62 @@ residual_terms_norm_vec_kernel(float* __restrict__ out32, T* __restrict__ out1, 
     if (out2) {
       const float4 g = *reinterpret_cast<const float4*>(gain2 + i);
       store4(out2 + at + i, make_float4(n.x * g.x, n.y * g.y, n.z * g.z, n.w * g.w));
+    }
+  }
+}
+
+__global__ void partial_residual_terms_norm_kernel(float* __restrict__ out32, __nv_bfloat16* __restrict__ out1,
+                                                   __nv_bfloat16* __restrict__ out2, const asb::PartialSums ps, float pf,
+                                                   const float* __restrict__ x, const Terms terms, const float* __restrict__ gain1,
+                                                   const float* __restrict__ gain2, int width, float eps) {
+  __shared__ float scratch[32];
+  const int t = blockIdx.x, i = threadIdx.x * 8;
+  const bool active = i < width;
+  const int slots = active ? asb::partial_slots(ps, i / asb::kPartialRows) : 0;
+  asb::pdl_wait();
+  asb::pdl_launch_dependents();
+  const size_t at = (size_t)t * width + i;
+  float s[8], y[8];
+#pragma unroll
+  for (int k = 0; k < 8; ++k) s[k] = y[k] = 0.f;
+  if (active) {
+    if (x) {
+      *reinterpret_cast<float4*>(s) = *reinterpret_cast<const float4*>(x + at);
+      *reinterpret_cast<float4*>(s + 4) = *reinterpret_cast<const float4*>(x + at + 4);
+    }
+#pragma unroll
+    for (int u = 0; u < kMaxTerms; ++u) {
+      if (u >= terms.n) break;
+      float v[8];
+      *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(terms.y[u] + at);
+      *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(terms.y[u] + at + 4);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) s[k] = fmaf(terms.f[u], v[k], s[k]);
+    }
+    asb::partial_sum<8>(ps, t, i, slots, y);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    s[k] = fmaf(pf, y[k], s[k]);
+    ss = fmaf(s[k], s[k], ss);
+  }
+  if (active) {
+    store4(out32 + at, make_float4(s[0], s[1], s[2], s[3]));
+    store4(out32 + at + 4, make_float4(s[4], s[5], s[6], s[7]));
+  }
+  if (!out1 && !out2) return;
+  const float inv = 1.f / sqrtf(asb::block_sum(ss, scratch) / (float)width + eps);
+  if (!active) return;
+#pragma unroll
+  for (int which = 0; which < 2; ++which) {
+    __nv_bfloat16* out = which ? out2 : out1;
+    const float* gain = which ? gain2 : gain1;
+    if (!out) continue;
+#pragma unroll
+    for (int k = 0; k < 8; k += 4) {
+      const float4 g = *reinterpret_cast<const float4*>(gain + i + k);
+      store4(out + at + k, make_float4(s[k] * inv * g.x, s[k + 1] * inv * g.y, s[k + 2] * inv * g.z, s[k + 3] * inv * g.w));
     }
   }
 }
@@ -253,6 +313,33 @@ extern "C" int asb_residual_terms_norm(float* out32, void* out1, void* out2, con
   ASB_DISPATCH_DTYPE(dtype, T, asb::launch(residual_terms_norm_kernel<T>, n, threads_for(width), width * sizeof(float),
                                            stream, out32, (T*)out1, (T*)out2, x, t, bias, gain1, gain2, width, eps));
   return asb::check_launch("residual_terms_norm");
+}
+
+// The form with a last term f y given as partial sums (asb_gemm_tcgen05 mode 3 on [n, K] x [width, K]); out1 and
+// out2 are bfloat16. Widths that are a multiple of 8 up to 8192, pointers 16-byte aligned.
+extern "C" int asb_partial_residual_terms_norm(float* out32, void* out1, void* out2, const float* ws, int max_slots, int bn,
+                                               int kb_per_tile, int num_tiles, int blocks, float f, const float* x, const float* y1,
+                                               const float* y2, const float* y3, const float* y4, float f1, float f2, float f3,
+                                               float f4, int terms, const float* gain1, const float* gain2, int n, int width,
+                                               float eps, cudaStream_t stream) {
+  if (n == 0) return 0;
+  if (width % 8 || width / 8 > 1024) return asb::fail("partial_residual_terms_norm: width %d must be a multiple of 8 up to 8192", width);
+  if (n > bn || num_tiles * asb::kPartialRows < width)
+    return asb::fail("partial_residual_terms_norm: %d tokens x %d columns do not fit the partial sums (%d x %d)", n, width, bn,
+                     num_tiles * asb::kPartialRows);
+  if (terms < 0 || terms > kMaxTerms) return asb::fail("partial_residual_terms_norm: %d terms, at most %d", terms, kMaxTerms);
+  if (!out32 || (out1 && !gain1) || (out2 && !gain2)) return asb::fail("partial_residual_terms_norm: outputs and their gains");
+  const Terms t = {{y1, y2, y3, y4}, {f1, f2, f3, f4}, terms};
+  uintptr_t all = (uintptr_t)out32 | (uintptr_t)out1 | (uintptr_t)out2 | (uintptr_t)x | (uintptr_t)gain1 | (uintptr_t)gain2 | (uintptr_t)ws;
+  for (int u = 0; u < terms; ++u) {
+    if (!t.y[u]) return asb::fail("partial_residual_terms_norm: term %d is missing", u);
+    all |= (uintptr_t)t.y[u];
+  }
+  if (all & 15) return asb::fail("partial_residual_terms_norm: pointers must be 16-byte aligned");
+  const asb::PartialSums ps = {ws, max_slots, bn, kb_per_tile, num_tiles, blocks};
+  asb::launch(partial_residual_terms_norm_kernel, n, ((width / 8) + 31) / 32 * 32, 0, stream, out32, (__nv_bfloat16*)out1,
+              (__nv_bfloat16*)out2, ps, f, x, t, gain1, gain2, width, eps);
+  return asb::check_launch("partial_residual_terms_norm");
 }
 
 extern "C" int asb_pair_embedding(float* out, const void* table, const void* pairs, const int* ids,

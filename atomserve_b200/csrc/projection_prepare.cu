@@ -145,6 +145,107 @@ projection_norm_rope_store_kernel(const ProjectionParams p) {
   }
 }
 
+// The usual form (bfloat16, pairs of halves): a thread keeps units of two vectors of eight entries in
+// registers from the projection to where they belong: the entries of a unit's first vector and those of its
+// second are pairs, or, past the rotated entries, neighbours that only take their norm. kPer: units a thread.
+template <int kPer>
+__global__ void __launch_bounds__(256)
+projection_norm_rope_store_units_kernel(const ProjectionParams p) {
+  using T = __nv_bfloat16;
+  extern __shared__ __align__(16) float cs[];  // [rotary_dim]: cosines, then sines
+  __shared__ float scratch[2][8];
+  const int qw = p.H * p.dim, kw = p.KV * p.dim, half = p.rotary_dim >> 1, turned = half >> 3, per = p.dim >> 4;
+  asb::pdl_wait();
+  asb::pdl_launch_dependents();
+  const int t = blockIdx.x, nwarps = blockDim.x >> 5;
+  const T* src = (const T*)p.proj + (size_t)t * p.stride + p.q_off;
+  const float position = (float)p.positions[t];
+  const int slot = p.slots ? p.slots[t] : -1;
+  const bool store = p.k_cache && slot >= 0;
+  const int units = (p.H + (store ? p.KV : 0)) * per;
+  float a[kPer][8], b[kPer][8];
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * blockDim.x;
+    if (i >= units) continue;
+    const int head = i / per, w = i - head * per;
+    const int e = w < turned ? w * 8 : p.rotary_dim + (w - turned) * 16;
+    load_row<T, 8>(src + head * p.dim + e, a[u]);
+    load_row<T, 8>(src + head * p.dim + e + (w < turned ? half : 8), b[u]);
+  }
+  for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(position * p.inv_freq[i], &cs[half + i], &cs[i]);
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * blockDim.x;
+    if (i >= units) continue;
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(a[u][j], a[u][j], fmaf(b[u][j], b[u][j], ss));
+    if (i < p.H * per) sq += ss;
+    else sk += ss;
+  }
+  sq = asb::warp_sum(sq);
+  sk = asb::warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    scratch[0][threadIdx.x >> 5] = sq;
+    scratch[1][threadIdx.x >> 5] = sk;
+  }
+  __syncthreads();  // (the angles too)
+  sq = sk = 0.f;
+  for (int w = 0; w < nwarps; ++w) {
+    sq += scratch[0][w];
+    sk += scratch[1][w];
+  }
+  const float inv_q = 1.f / sqrtf(sq / (float)qw + p.eps), inv_k = 1.f / sqrtf(sk / (float)kw + p.eps);
+  const size_t page = store ? slot / p.bs : 0, off = store ? slot % p.bs : 0;
+#pragma unroll
+  for (int u = 0; u < kPer; ++u) {
+    const int i = threadIdx.x + u * blockDim.x;
+    if (i >= units) continue;
+    const int head = i / per, w = i - head * per;
+    const bool query = head < p.H;
+    const int e = w < turned ? w * 8 : p.rotary_dim + (w - turned) * 16, f = e + (w < turned ? half : 8);
+    const float* gain = query ? p.q_gain + head * p.dim : p.k_gain + (head - p.H) * p.dim;
+    const float inv = query ? inv_q : inv_k;
+    float ga[8], gb[8];
+#pragma unroll
+    for (int j = 0; j < 8; j += 4) {
+      *reinterpret_cast<float4*>(ga + j) = *reinterpret_cast<const float4*>(gain + e + j);
+      *reinterpret_cast<float4*>(gb + j) = *reinterpret_cast<const float4*>(gain + f + j);
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      a[u][j] *= inv * ga[j];
+      b[u][j] *= inv * gb[j];
+    }
+    if (w < turned) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float c = cs[e + j], s = cs[half + e + j], x = a[u][j], y = b[u][j];
+        a[u][j] = x * c - y * s;
+        b[u][j] = y * c + x * s;
+      }
+    }
+    T* dst = query ? (T*)p.q_out + ((size_t)t * p.H + head) * p.hd : (T*)p.k_cache + ((page * p.KV + head - p.H) * p.bs + off) * p.hd;
+    store_row<T, 8>(dst + e, a[u]);
+    store_row<T, 8>(dst + f, b[u]);
+  }
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  const int kz = (p.hd - p.dim) >> 3, per_v = p.hd >> 3;
+  for (int i = threadIdx.x; i < (p.H + (store ? p.KV : 0)) * kz; i += blockDim.x) {  // zeros behind queries and keys
+    const int head = i / kz, e = p.dim + i % kz * 8;
+    T* dst = head < p.H ? (T*)p.q_out + ((size_t)t * p.H + head) * p.hd : (T*)p.k_cache + ((page * p.KV + head - p.H) * p.bs + off) * p.hd;
+    *reinterpret_cast<uint4*>(dst + e) = zero;
+  }
+  if (!store) return;
+  for (int i = threadIdx.x; i < p.KV * per_v; i += blockDim.x) {
+    const int head = i / per_v, e = (i - head * per_v) * 8;
+    *reinterpret_cast<uint4*>((T*)p.v_cache + ((page * p.KV + head) * p.bs + off) * p.hd + e) =
+        e < p.vdim ? *reinterpret_cast<const uint4*>(src + qw + kw + head * p.vdim + e) : zero;
+  }
+}
+
 template <typename T, int VEC>
 int launch(const ProjectionParams& p, int T_, cudaStream_t stream) {
   const size_t smem = sizeof(float) * ((size_t)(p.H + p.KV) * p.dim + p.rotary_dim);
@@ -176,6 +277,16 @@ extern "C" int asb_projection_norm_rope_store(const void* proj, int stride, int 
   const bool aligned = (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0;
   const int vec = dtype == asb::kBFloat16 ? 8 : 4;
   if (aligned && dim % vec == 0 && vdim % vec == 0 && stride % vec == 0 && q_off % vec == 0) {
+    const int units = (H + KV) * (dim / 16);
+    if (dtype == asb::kBFloat16 && !interleaved && dim % 16 == 0 && rotary_dim % 16 == 0 && units <= 1024 &&
+        (((uintptr_t)q_gain | (uintptr_t)k_gain) & 15) == 0) {
+      const int threads = units >= 256 ? 256 : (units + 31) / 32 * 32;
+      const size_t smem = sizeof(float) * (rotary_dim > 0 ? rotary_dim : 1);
+      if (units <= 256) asb::launch(projection_norm_rope_store_units_kernel<1>, T_, threads, smem, stream, p);
+      else if (units <= 512) asb::launch(projection_norm_rope_store_units_kernel<2>, T_, threads, smem, stream, p);
+      else asb::launch(projection_norm_rope_store_units_kernel<4>, T_, threads, smem, stream, p);
+      return asb::check_launch("projection_norm_rope_store");
+    }
     if (dtype == asb::kBFloat16) return launch<__nv_bfloat16, 8>(p, T_, stream);
     if (dtype == asb::kFloat32) return launch<float, 4>(p, T_, stream);
   }

@@ -107,6 +107,7 @@ _SIGNATURES = {
     "asb_prefill_attention_tcgen05_masked": [_P] * 8 + [_I] * 10 + [_F, _F, _P, _P],
     # layers whose two sublayers read one stream; a hashed table of token pairs; a product over two streams
     "asb_residual_terms_norm": [_P] * 8 + [_F] * 4 + [_I] + [_P] * 3 + [_I, _I, _F, _I, _P],
+    "asb_partial_residual_terms_norm": [_P] * 4 + [_I] * 5 + [_F] + [_P] * 5 + [_F] * 4 + [_I] + [_P] * 2 + [_I, _I, _F, _P],
     "asb_pair_embedding": [_P] * 8 + [_I] * 8 + [_P, _P],
     "asb_concat_cast": [_P, _P, _P, _I, _I, _I, _P],
     # parallel residual streams; scores mixed across heads, kept first positions; experts without a gate

@@ -7,6 +7,7 @@ from __future__ import annotations
 import torch
 
 from atomserve_b200.ops.library import KernelLibraryError, check, dtype_code, lib, ptr, require_cuda, stream
+from atomserve_b200.ops.linear import PartialSums
 
 
 def _rows32(t: torch.Tensor | None, name: str, shape: tuple) -> None:
@@ -14,12 +15,16 @@ def _rows32(t: torch.Tensor | None, name: str, shape: tuple) -> None:
         raise KernelLibraryError(f"{name} must be contiguous float32 {list(shape)}, got {t.dtype} {tuple(t.shape)}")
 
 
-def residual_terms_norm(x: torch.Tensor | None, terms: list[tuple[torch.Tensor, float]], gain1: torch.Tensor | None,
+def residual_terms_norm(x: torch.Tensor | None, terms: list[tuple[torch.Tensor | PartialSums, float]], gain1: torch.Tensor | None,
                         gain2: torch.Tensor | None, eps: float, dtype: torch.dtype, *, bias: torch.Tensor | None = None,
                         want_stream: bool = True) -> tuple[torch.Tensor | None, torch.Tensor | None, torch.Tensor | None]:  # fmt: skip
     """s = x + sum of f y over the (y, f) of `terms` (at most four) + bias, x and bias optional (float32
     [n, width]; bias [width]), and its two norms N(s) gain1, N(s) gain2 in `dtype`,
-    N(s) = s / sqrt(mean(s^2) + eps). Returns (s or None, first norm or None, second norm or None)."""
+    N(s) = s / sqrt(mean(s^2) + eps). The last term may be the partial sums of a product
+    (`linear_for_stream`), which the kernel then adds up itself. Returns (s or None, first norm or None,
+    second norm or None)."""
+    if terms and isinstance(terms[-1][0], PartialSums):
+        return _with_partial_sums(x, terms[:-1], *terms[-1], gain1, gain2, eps, dtype, bias, want_stream)
     first = x if x is not None else (terms[0][0] if terms else None)
     if first is None or len(terms) > 4:
         raise KernelLibraryError(f"residual_terms_norm: {len(terms)} terms" if terms else "residual_terms_norm: nothing to add")
@@ -38,6 +43,26 @@ def residual_terms_norm(x: torch.Tensor | None, terms: list[tuple[torch.Tensor, 
     fs = [float(f) for _, f in terms] + [0.0] * (4 - len(terms))
     check(lib().asb_residual_terms_norm(ptr(out32), ptr(out1), ptr(out2), ptr(x), *ys, *fs, len(terms), ptr(bias), ptr(gain1),
                                         ptr(gain2), n, width, float(eps), code, stream()))  # fmt: skip
+    return out32, out1, out2
+
+
+def _with_partial_sums(x, terms, product: PartialSums, factor: float, gain1, gain2, eps: float, dtype, bias, want_stream):
+    n, width = product.tokens, product.columns
+    if bias is not None or not want_stream or dtype != torch.bfloat16 or len(terms) > 4:
+        raise KernelLibraryError("residual_terms_norm: partial sums join a stream that is kept, beside bfloat16 products, without a bias")
+    require_cuda(x, gain1, gain2, *(y for y, _ in terms))
+    for t in (x, *(y for y, _ in terms)):
+        _rows32(t, "a term", (n, width))
+    for t in (gain1, gain2):
+        _rows32(t, "gain", (width,))
+    device = product.workspace.device
+    out32 = torch.empty(n, width, device=device, dtype=torch.float32)
+    out1 = torch.empty(n, width, device=device, dtype=dtype) if gain1 is not None else None
+    out2 = torch.empty(n, width, device=device, dtype=dtype) if gain2 is not None else None
+    ys = [ptr(y) for y, _ in terms] + [None] * (4 - len(terms))
+    fs = [float(f) for _, f in terms] + [0.0] * (4 - len(terms))
+    check(lib().asb_partial_residual_terms_norm(ptr(out32), ptr(out1), ptr(out2), ptr(product.workspace), *product.layout(), float(factor),
+                                                ptr(x), *ys, *fs, len(terms), ptr(gain1), ptr(gain2), n, width, float(eps), stream()))  # fmt: skip
     return out32, out1, out2
 
 

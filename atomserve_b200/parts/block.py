@@ -152,7 +152,8 @@ class ParallelResidualBlock(PostNormBlock):
     as several float32 terms with a factor each. The kernel that adds a layer's outputs also
     norms the sum twice for the next block of this kind, so the pair (N1 x, N2 x) travels from
     block to block in the place where pre-norm blocks hand on their normed input. Sublayers give
-    float32 outputs (`forward_for_stream` must not leave partial sums: two products are added)."""
+    float32 outputs; a feed-forward that ends in a plain product (`ends_in_product`) runs last and may
+    leave it as partial sums, which that kernel adds up (one product only: they share a workspace)."""
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         super().load(tensors)
@@ -171,7 +172,8 @@ class ParallelResidualBlock(PostNormBlock):
         several = getattr(self.mixer, "forward_terms", None)
         terms = several(h1, ctx, cache, write_cache) if several is not None else [(self.mixer.forward(h1, None, ctx, cache, write_cache), 1.0)]
         if self.has_feed_forward:
-            terms.append((self.feed_forward.forward(h2, None, ctx), 1.0))
+            plain = getattr(self.feed_forward, "ends_in_product", False)
+            terms.append((self.feed_forward.forward_for_stream(h2, ctx) if plain else self.feed_forward.forward(h2, None, ctx), 1.0))
         terms = [(y, f * self.mult) for y, f in terms]
         owner = getattr(then, "block_norms", None) if then is not None else None
         if owner is None:  # the last block, or one of another kind next: the sum alone

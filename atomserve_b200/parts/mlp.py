@@ -89,6 +89,11 @@ class GatedMLP(FeedForward):
             self.gate_up_bias = (torch.stack([b_gate, b_up], dim=1).reshape(-1) if self.fused else torch.cat([b_gate, b_up])).contiguous()
             self.output_bias = tensors[p + "down.b"]
 
+    @property
+    def ends_in_product(self) -> bool:
+        """Whether `forward_for_stream` is the whole of `forward` (there is no output bias to add)."""
+        return not self.biases
+
     def inner(self, h: torch.Tensor) -> torch.Tensor:
         if self.fused:
             return ops.linear_glu(h, self.gate_up, self.gate_up_bias, self.activation)

@@ -1182,6 +1182,181 @@ def time_lidizen(widths: list[int], layers: int, steps: int, warmup: int, pk: di
         print(json.dumps(line), flush=True)
 
 
+# ---- the Vilulix design beside Zogepel at equal width (`--only vilulix`) --------------------------
+
+def vilulix_shape(width: int, layers: int) -> dict:
+    """Layer sizes that resemble a served model's: a matrix memory with keys half as wide as values;
+    attention over a latent of 512 + 64 with queries through a latent of three quarters of the width;
+    attention with heads of 128 in a window of 1,024, four query heads a kv head, beside a delta rule
+    with heads of 128 x 128, two a q/k head, four taps; in turn, each with a feed-forward of four times
+    the width (every layer runs once: a loop would repeat what one pass does)."""
+    heads = width // 128
+    out = []
+    for i in range(layers):
+        if i % 3 == 0:
+            layer = dict(type="mlstm", mixer=dict(heads=heads, dim=64, vdim=128, gate_cap=15.0))
+        elif i % 3 == 1:
+            layer = dict(type="latent_attention", mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=3 * width // 4,
+                                                             scale=192 ** -0.5, rot=dict(base=10000.0, dims=64)))
+        else:
+            left = dict(heads=heads, kv_heads=max(heads // 4, 1), dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024),
+                        rot=dict(base=1000000.0, dims=128))
+            right = dict(heads=heads, kv_heads=max(heads // 2, 1), dim=128, vdim=128, conv=4)
+            layer = dict(type="parallel", mixer=dict(left=left, right=right, left_scale=1.0, right_scale=0.8))
+        out.append(dict(layer, mlp=dict(kind="dense", ff=4 * width)))
+    return dict(architecture="Vilulix", vocab=32000, width=width, layers=out, norm=dict(eps=1e-6), logit_softcap=30.0)
+
+
+def time_vilulix(widths: list[int], layers: int, steps: int, warmup: int, pk: dict) -> None:
+    """Prefill and decode of a Vilulix model and of a Zogepel model of the same width and depth (random
+    weights), through the step function, and the design's own kernels one by one against their
+    rooflines beside the like kernels of the other models."""
+    import torch
+
+    from atomserve_b200 import ops
+
+    timed, model_times = design_timers(steps, warmup)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")  # noqa: E731
+    bw, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    bf = torch.bfloat16
+    for width in widths:
+        line = {"only": "vilulix", "width": width, "layers": layers, "peaks": pk["source"],
+                "vilulix": model_times(vilulix_shape(width, layers), 32000), "zogepel": model_times(zogepel_shape(width, layers), 32000)}
+        kern = {}
+        T, B, ctx, bs = PROMPT_TOKENS, 64, PROMPT_TOKENS, BLOCK_SIZE
+        H, hd = width // 128, 128
+        one, each = (i32([0]), i32([0, T])), (i32(list(range(B))), i32(list(range(B + 1))))
+        positions, slots = i32(list(range(T))), i32(list(range(T)))
+
+        # the recurrences, float32 on CUDA cores: 6 floating-point operations a state entry and token for the delta
+        # rule (S^T k, S^T q and the update), 4 for the others; decode: states read and written
+        D, V, G = 128, 128, max(H // 2, 1)
+        x = torch.randn(T, 2 * G * D + H * V, device="cuda", dtype=bf)
+        z, zero = torch.randn(T, 2 * H, device="cuda"), torch.zeros(H, device="cuda")
+        state = torch.zeros(B, H, D, V, device="cuda")
+        for name, rows, (at, starts), n, lens in (("prefill", T, one, 1, [T]), ("decode_b64", B, each, B, [1] * B)):
+            plan = ops.plan_delta(lens, H, D, V, x.device)
+            ms = timed(lambda: ops.delta_rule(x[:rows], 0, G * D, 2 * G * D, z[:rows], 0, H, zero, zero, state, at, starts, n, kv_heads=G, plan=plan))
+            kern[f"delta_rule_{name}"] = ({"ms": round(ms, 4), "gflops": round(6.0 * T * H * D * V / ms / 1e6, 1), "note": "float32 CUDA cores"}
+                                          if rows == T else {"ms": round(ms, 4), "hbm_frac": round(2.0 * B * H * D * V * 4 / (ms * 1e-3) / bw, 3)})  # fmt: skip
+        Dm = 64
+        proj = torch.randn(T, 2 * H * Dm + 2 * H * V, device="cuda", dtype=bf)
+        mstate, norm_state, top = torch.zeros(B, H, Dm, V, device="cuda"), torch.zeros(B, H, Dm, device="cuda"), torch.zeros(B, H, device="cuda")
+        for name, rows, (at, starts), n, seg in (("prefill", T, one, 1, ops.plan_segments([T], x.device)), ("decode_b64", B, each, B, None)):
+            def memory():
+                a, b, _ = ops.capped_gates_scan(z[:rows], 0, H, H, zero, zero, 15.0, top, at, starts, n)
+                return ops.linear_recurrence(proj[:rows], 0, H * Dm, 2 * H * Dm, mstate, at, starts, n, token_decay=a, token_gain=b,
+                                             norm_state=norm_state, q_scale=Dm ** -0.5, segments=seg)  # fmt: skip
+
+            ms = timed(memory, 8)
+            kern[f"matrix_memory_{name}"] = ({"ms": round(ms, 4), "gflops": round(4.0 * T * H * Dm * (V + 1) / ms / 1e6, 1), "note": "float32 CUDA cores"}
+                                             if rows == T else {"ms": round(ms, 4), "hbm_frac": round(2.0 * B * H * Dm * (V + 1) * 4 / (ms * 1e-3) / bw, 3)})  # fmt: skip
+        # the short convolutions with their state, beside Tigesun's
+        C, K = 2 * G * D + H * V, 4
+        wide = torch.randn(T, C + H * V + H, device="cuda", dtype=bf)
+        taps, held, bias = torch.randn(C, K, device="cuda"), torch.zeros(B, K - 1, C, device="cuda"), torch.zeros(C, device="cuda")
+        for name, rows, (at, starts), n, lens in (("prefill", T, one, 1, [T]), ("decode_b64", B, each, B, [1] * B)):
+            moved = rows * C * 4 + n * (K - 1) * C * 8
+            ms = timed(lambda: ops.causal_conv_silu(wide[:rows], 0, taps, held, at, starts, n, lens))
+            kern[f"causal_conv_silu_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(moved / (ms * 1e-3) / bw, 3)}
+
+            def steps_and_state():
+                ops.conv_steps(wide[:rows], 0, C, taps, bias, held, zero, zero, at, starts, n)
+                ops.conv_state_update(held, wide[:rows], 0, at, starts, n)
+
+            ms = timed(steps_and_state)
+            kern[f"conv_steps_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(moved / (ms * 1e-3) / bw, 3)}
+        o, gate = torch.randn(T, H * V, device="cuda"), wide[:, C : C + H * V]
+        g2 = torch.ones(H * V, device="cuda")
+        for name, act in (("head_norm_silu_gate", "silu"), ("head_norm_sigmoid_gate", "sigmoid")):
+            ms = timed(lambda: ops.head_norm_gate(o, gate, H, gain=g2, eps=1e-6, gate_activation=act))
+            kern[name] = {"ms": round(ms, 4), "hbm_frac": round(T * H * V * 8 / (ms * 1e-3) / bw, 3)}
+        del wide, o, gate, state, mstate
+
+        # attention in a window of 1,024 with the fixed term in its denominator, beside the same window without
+        KV, window = max(H // 4, 1), 1024
+        pages_per = ctx // bs
+        tables, t1 = i32([[r * pages_per + j for j in range(pages_per)] for r in range(B)]), i32([list(range(pages_per))])
+        starts, at = i32(list(range(B + 1))), i32([ctx - 1] * B)
+        k_pages = torch.randn(B * pages_per, KV, bs, hd, device="cuda", dtype=bf)
+        v_pages = torch.randn_like(k_pages)
+        sink = torch.zeros(H, device="cuda")
+        q, qp = torch.randn(B, H, hd, device="cuda", dtype=bf), torch.randn(T, H, hd, device="cuda", dtype=bf)
+        seen = sum(min(t + 1, window) for t in range(T))
+        for name, sk in (("window_attention", sink), ("window_attention_no_sink", None)):
+            ms = timed(lambda: ops.paged_attention(q, k_pages, v_pages, tables, starts, at, num_requests=B, max_context=ctx, window=window,
+                                                   scale=0.088, host_q_lens=[1] * B, sink=sk))  # fmt: skip
+            kern[f"{name}_decode_b64"] = {"ms": round(ms, 4), "hbm_frac": round(2.0 * B * window * KV * hd * 2 / (ms * 1e-3) / bw, 3)}
+            ms = timed(lambda: ops.paged_attention(qp, k_pages, v_pages, t1, i32([0, T]), i32([0]), num_requests=1, max_context=T,
+                                                   window=window, scale=0.088, host_q_lens=[T], sink=sk), 4)  # fmt: skip
+            kern[f"{name}_prefill"] = {"ms": round(ms, 3), "tc_frac": round(4.0 * seen * H * hd / (ms * 1e-3) / tf, 4)}
+        # between projection and attention: norm over the projection, rotation, page write, beside the norm per head
+        inv = (1.0 / 1000000.0 ** (torch.arange(0, hd, 2, dtype=torch.float32) / hd)).cuda()
+        gq, gk, g1 = torch.ones(H * hd, device="cuda"), torch.ones(KV * hd, device="cuda"), torch.ones(hd, device="cuda")
+        for name, rows in (("prefill", T), ("decode_b64", B)):
+            qkv = torch.randn(rows, (H + 2 * KV) * hd, device="cuda", dtype=bf)
+            moved = rows * (2 * H + 4 * KV) * hd * 2
+            ms = timed(lambda: ops.projection_norm_rope_store(qkv, 0, H, KV, hd, hd, hd, positions[:rows], gq, gk, 1e-6, inv_freq=inv, rotary_dim=hd,
+                                                              slots=slots[:rows], k_cache=k_pages, v_cache=v_pages))  # fmt: skip
+            kern[f"projection_norm_rope_store_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(moved / (ms * 1e-3) / bw, 3)}
+            ms = timed(lambda: ops.qk_norm_rope_store(qkv, H, KV, hd, positions[:rows], q_gain=g1, k_gain=g1, eps=1e-6, inv_freq=inv,
+                                                      rotary_dim=hd, slots=slots[:rows], k_cache=k_pages, v_cache=v_pages))  # fmt: skip
+            kern[f"qk_norm_rope_store_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(moved / (ms * 1e-3) / bw, 3)}
+        del k_pages, v_pages
+
+        # attention over the latent: the kernels Gefilix runs, with this design's queries, rotation and gate beside them
+        R, Rt, Qr = 512, 64, 3 * width // 4
+        lat_pages = torch.randn(B * pages_per, 1, bs, R + Rt, device="cuda", dtype=bf)
+        lat_inv = (1.0 / 10000.0 ** (torch.arange(0, Rt, 2, dtype=torch.float32) / Rt)).cuda()
+        uk, uv = torch.randn(H, R, hd, device="cuda", dtype=bf), torch.randn(H, hd, R, device="cuda", dtype=bf)
+        for name, rows in (("prefill", T), ("decode_b64", B)):
+            q_lat = torch.randn(rows, H, R + Rt, device="cuda")
+            many = name == "prefill"
+            ms = timed(lambda: ops.latent_attention(q_lat, lat_pages, t1 if many else tables, i32([0, T]) if many else starts, i32([0]) if many else at,
+                                                    rank=R, num_requests=1 if many else B, max_context=ctx, scale=0.07), 4)  # fmt: skip
+            kern[f"latent_attention_{name}"] = {"ms": round(ms, 4), **({"tc_frac": round(2.0 * T * T / 2 * H * (2 * R + Rt) / (ms * 1e-3) / tf, 4)} if many else
+                                                                      {"hbm_frac": round(B * ctx * (R + Rt) * 2 / (ms * 1e-3) / bw, 3)})}  # fmt: skip
+            down = torch.randn(rows, Qr + R + Rt + H * hd, device="cuda", dtype=bf)
+            queries = torch.randn(rows, H * (hd + Rt), device="cuda", dtype=bf)
+            gain = torch.ones(R, device="cuda")
+            for half in (True, False):
+                ms = timed(lambda: ops.latent_prepare(down, 0, Qr, q_lat, lat_pages, gain, lat_inv, positions[:rows], slots[:rows], heads=H, dim=hd, rank=R,
+                                                      rot=Rt, rot_dims=Rt, eps=1e-6, queries=queries, half_pairs=half))  # fmt: skip
+                kern[f"latent_prepare_{'half' if half else 'neighbour'}_pairs_{name}"] = {
+                    "ms": round(ms, 4), "hbm_frac": round(rows * (H * Rt * 6 + (R + Rt) * 4) / (ms * 1e-3) / bw, 3)}
+            gr = torch.ones(Qr, device="cuda")
+            ms = timed(lambda: ops.rms_norm(down[:, :Qr], gr, 1e-6))
+            kern[f"query_latent_norm_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * Qr * 4 / (ms * 1e-3) / bw, 3)}
+            ms = timed(lambda: ops.head_matmul(queries.view(rows, H, hd + Rt)[:, :, :hd], uk, q_lat[:, :, :R], w_is_nk=True))
+            kern[f"queries_into_latent_{name}"] = {"ms": round(ms, 4), "tc_frac": round(2.0 * rows * H * hd * R / (ms * 1e-3) / tf, 4)}
+            mixed, out = q_lat[:, :, :R].contiguous(), torch.empty(rows, H, hd, device="cuda", dtype=bf)
+            for gname, gt in (("element_gates", down[:, -H * hd :]), ("head_gates", down[:, -H:])):
+                ms = timed(lambda: ops.head_matmul(mixed, uv, out, gate=gt, w_is_nk=True))
+                kern[f"values_out_of_latent_{gname}_{name}"] = {"ms": round(ms, 4), "tc_frac": round(2.0 * rows * H * hd * R / (ms * 1e-3) / tf, 4)}
+            del down, q_lat, queries, mixed, out
+        del lat_pages
+
+        # the sum of a layer's outputs and both norms of the next one: three terms (a layer of two mixers), two, and
+        # Gefilix's one with one norm
+        gain = torch.ones(width, device="cuda")
+        for name, rows in (("prefill", T), ("decode_b64", B)):
+            xs = [torch.randn(rows, width, device="cuda") for _ in range(4)]
+            for n in (3, 2):
+                ms = timed(lambda: ops.residual_terms_norm(xs[0], [(y, 0.9) for y in xs[1 : n + 1]], gain, gain, 1e-6, bf))
+                kern[f"residual_terms_norm_{n}_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * width * (4 * n + 12) / (ms * 1e-3) / bw, 3)}
+            ms = timed(lambda: ops.scaled_add_rms_norm(xs[0], xs[1], 1.0, gain, 1e-6, bf))
+            kern[f"scaled_add_rms_norm_{name}"] = {"ms": round(ms, 4), "hbm_frac": round(rows * width * 14 / (ms * 1e-3) / bw, 3)}
+            # the feed-forward's fused products
+            h, w_gu = torch.randn(rows, width, device="cuda", dtype=bf), torch.randn(8 * width, width, device="cuda", dtype=bf)
+            for fname, fn in (("gate_up_silu", lambda: ops.linear_glu(h, w_gu, None, "silu")), ("gate_up_swiglu", lambda: ops.linear_swiglu(h, w_gu))):
+                ms = timed(fn, 8)
+                kern[f"{fname}_{name}"] = {"ms": round(ms, 4), "tc_frac": round(2.0 * rows * width * 8 * width / (ms * 1e-3) / tf, 4),
+                                           "hbm_frac": round(8 * width * width * 2 / (ms * 1e-3) / bw, 3)}  # fmt: skip
+            del h, w_gu
+        line["kernels"] = kern
+        print(json.dumps(line), flush=True)
+
+
 def tigesun_inner(width: int, ff: int, w_gu, b_gu):
     """A gated feed-forward part holding the given stacked gate and up rows ([2 ff, width], gate first)."""
     import torch
@@ -1249,7 +1424,7 @@ def main() -> int:
                         help="fewer layers than the model has (same layer sizes), where time or memory needs it")  # fmt: skip
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    parser.add_argument("--only", choices=["decode", "prefill", "gemm", "serve", "attention", "sampling", "designs", "zogepel", "tigesun", "nipurax", "lidizen"], help="time just this (for profiling small cases and the other shapes)")
+    parser.add_argument("--only", choices=["decode", "prefill", "gemm", "serve", "attention", "sampling", "designs", "zogepel", "tigesun", "nipurax", "lidizen", "vilulix"], help="time just this (for profiling small cases and the other shapes)")
     parser.add_argument("--shape", default="8b", choices=sorted(SHAPES), help="with --only decode/prefill/serve: layer sizes of Qwen3-8B, -14B or -32B")
     parser.add_argument("--context", type=int, default=PROMPT_TOKENS, help="with --only decode: tokens each request holds when decoding starts")
     parser.add_argument("--requests", type=int, default=32, help="with --only serve: requests submitted at once")
@@ -1257,7 +1432,7 @@ def main() -> int:
     parser.add_argument("--budget", type=int, default=512, help="with --only serve: the scheduler's token budget per step")
     parser.add_argument("--gemm-shape", default="all", help="with --only gemm: qkv, o, gate_up, down, lm_head or all")
     parser.add_argument("--gemm-tokens", default="1,8,64,2048", help="with --only gemm: token counts, comma-separated")
-    parser.add_argument("--widths", default="2048,4096", help="with --only designs, zogepel, tigesun, nipurax or lidizen: model widths, comma-separated")
+    parser.add_argument("--widths", default="2048,4096", help="with --only designs, zogepel, tigesun, nipurax, lidizen or vilulix: model widths, comma-separated")
     parser.add_argument("--timeline", action="store_true", help="with --only gemm: where a decode-size call's time goes")
     args = parser.parse_args()
     args.layers_given = any(a == "--layers" or a.startswith("--layers=") for a in sys.argv[1:])
@@ -1294,6 +1469,9 @@ def main() -> int:
         return 0
     if args.only == "lidizen":
         time_lidizen([int(w) for w in args.widths.split(",")], args.layers if args.layers_given else 4, max(args.steps // 4, 8), warmup, pk)
+        return 0
+    if args.only == "vilulix":
+        time_vilulix([int(w) for w in args.widths.split(",")], args.layers if args.layers_given else 4, max(args.steps // 4, 8), warmup, pk)
         return 0
     if args.only == "gemm" and args.timeline:
         gemm_timelines(args.gemm_shape, [int(t) for t in args.gemm_tokens.split(",")])

@@ -57,6 +57,31 @@ def test_sum_of_terms_and_both_norms_of_it(dtype, d):
         ops.residual_terms_norm(x.cuda(), [(y.cuda(), 1.0) for y in ys + ys[:1]], None, None, 0.0, dtype)
 
 
+def test_sum_whose_last_term_is_a_products_partial_sums():
+    """With few tokens a layer's last product stays as the GEMM's partial sums and the sum's kernel adds
+    them up: the finished product as a term, up to the order in which a row's sums are formed."""
+    from atomserve_b200 import ops
+    from atomserve_b200.ops.linear import PartialSums
+
+    g = torch.Generator().manual_seed(4)
+    met = 0
+    for T, d, K in ((1, 256, 512), (5, 336, 1024), (8, 2048, 2048), (33, 256, 392)):
+        inner = torch.randn(T, K, generator=g).bfloat16().cuda()
+        w = (torch.randn(d, K, generator=g) * K**-0.5).bfloat16().cuda()
+        x, y1, y2 = (torch.randn(T, d, generator=g).cuda() for _ in range(3))
+        g1, g2 = ((1 + 0.1 * torch.randn(d, generator=g)).cuda() for _ in range(2))
+        for terms, gains in (([], (g1, g2)), ([(y1, 0.7)], (g1, None)), ([(y1, -1.5), (y2, 0.4)], (g1, g2)), ([(y1, 1.0)], (None, None))):
+            whole = ops.residual_terms_norm(x, [*terms, (ops.linear(inner, w, out_dtype=torch.float32), 1.3)], *gains, EPS, torch.bfloat16)
+            y = ops.linear_for_stream(inner, w)
+            met += isinstance(y, PartialSums)
+            fused = ops.residual_terms_norm(x, [*terms, (y, 1.3)], *gains, EPS, torch.bfloat16)
+            assert float((whole[0] - fused[0]).abs().max() / whole[0].abs().max()) < 2e-6, (T, d, K)
+            for a, b, gain in zip(whole[1:], fused[1:], gains):
+                assert (a is None) == (b is None) == (gain is None)
+                assert gain is None or bool(((a.float() - b.float()).abs() <= 2.0**-7 * a.float().abs() + 1e-30).all()), (T, d, K)
+    assert met, "no shape ran with partial sums"
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_gains_around_zero_and_the_opening_of_a_pass(dtype):
     from atomserve_b200.parts import PartSpec, build_part
