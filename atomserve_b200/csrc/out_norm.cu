@@ -210,36 +210,46 @@ __global__ void projection_norm_store_kernel(T* __restrict__ q_out, const T* __r
   }
 }
 
-// One block per request, a warp per head (in turn), 32 tokens at a time: a lane turns its token's
-// pre-activations into log gates; the running maximum is a scan of the maps x -> max(x + f, i),
-// which compose as (f1, i1) then (f2, i2) = (f1 + f2, max(i1 + f2, i2)): five shuffle steps give
-// every lane the map of the group's tokens up to its own, applied to the maximum the group
-// starts from. Within a group the sums of f are grouped differently from token-by-token steps:
-// equal beyond rounding.
-__global__ void capped_gates_scan_kernel(float* __restrict__ decay, float* __restrict__ gain, float* __restrict__ top_out,
-                                         const float* __restrict__ z, int z_stride, int i_off, int f_off,
-                                         const float* __restrict__ i_bias, const float* __restrict__ f_bias,
-                                         float* __restrict__ top_state, const int* __restrict__ state_slots,
-                                         const int* __restrict__ req_q_start, int H, float cap) {
+// One warp per (request, head), 32 tokens at a time: a lane turns its token's pre-activations into
+// log gates; the running maximum is a scan of the maps x -> max(x + f, i), which compose as (f1, i1)
+// then (f2, i2) = (f1 + f2, max(i1 + f2, i2)): five shuffle steps give every lane the map of the
+// group's tokens up to its own, applied to the maximum the group starts from. Within a group the
+// sums of f are grouped differently from token-by-token steps: equal beyond rounding. Four groups'
+// pre-activations are fetched and turned into gates together before the chain through them is walked.
+__global__ void __launch_bounds__(32)
+capped_gates_scan_kernel(float* __restrict__ decay, float* __restrict__ gain, float* __restrict__ top_out,
+                         const float* __restrict__ z, int z_stride, int i_off, int f_off,
+                         const float* __restrict__ i_bias, const float* __restrict__ f_bias,
+                         float* __restrict__ top_state, const int* __restrict__ state_slots,
+                         const int* __restrict__ req_q_start, int H, float cap) {
+  constexpr int kGroups = 4;
   asb::pdl_wait();
   asb::pdl_launch_dependents();
-  const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+  const int r = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
   const int lo = req_q_start[r], hi = req_q_start[r + 1];
   const float inv_cap = 1.f / cap;
-  for (int h = warp; h < H; h += nwarps) {
-    float* ts = top_state + (size_t)state_slots[r] * H + h;
-    float top = *ts;  // the maximum before the group's first token (the same in every lane)
-    const float bi = i_bias[h], bf = f_bias[h];
-    for (int t0 = lo; t0 < hi; t0 += 32) {
-      const int t = t0 + lane;
-      const bool real = t < hi;
-      float f = 0.f, i = -INFINITY;  // the identity map for lanes past the end
-      if (real) {
-        const float u = cap * tanhf((z[(size_t)t * z_stride + f_off + h] + bf) * inv_cap);
-        f = fminf(u, 0.f) - log1pf(expf(-fabsf(u)));  // log sigmoid(u)
-        i = cap * tanhf((z[(size_t)t * z_stride + i_off + h] + bi) * inv_cap);
-      }
-      float F = f, I = i;
+  float* ts = top_state + (size_t)state_slots[r] * H + h;
+  float top = *ts;  // the maximum before the group's first token (the same in every lane)
+  const float bi = i_bias[h], bf = f_bias[h];
+  for (int t0 = lo; t0 < hi; t0 += 32 * kGroups) {
+    float f[kGroups], i[kGroups];
+#pragma unroll
+    for (int g = 0; g < kGroups; ++g) {
+      const int t = t0 + 32 * g + lane;
+      f[g] = t < hi ? z[(size_t)t * z_stride + f_off + h] : 0.f;
+      i[g] = t < hi ? z[(size_t)t * z_stride + i_off + h] : 0.f;
+    }
+#pragma unroll
+    for (int g = 0; g < kGroups; ++g) {
+      const bool real = t0 + 32 * g + lane < hi;
+      const float u = cap * tanhf((f[g] + bf) * inv_cap);
+      f[g] = real ? fminf(u, 0.f) - log1pf(expf(-fabsf(u))) : 0.f;  // log sigmoid(u); past the end the identity map
+      i[g] = real ? cap * tanhf((i[g] + bi) * inv_cap) : -INFINITY;
+    }
+#pragma unroll
+    for (int g = 0; g < kGroups; ++g) {
+      if (t0 + 32 * g >= hi) break;
+      float F = f[g], I = i[g];
 #pragma unroll
       for (int off = 1; off < 32; off <<= 1) {
         const float pF = __shfl_up_sync(0xffffffffu, F, off), pI = __shfl_up_sync(0xffffffffu, I, off);
@@ -251,16 +261,17 @@ __global__ void capped_gates_scan_kernel(float* __restrict__ decay, float* __res
       const float mine = fmaxf(top + F, I);
       float before = __shfl_up_sync(0xffffffffu, mine, 1);
       if (lane == 0) before = top;
-      if (real) {
+      const int t = t0 + 32 * g + lane;
+      if (t < hi) {
         const size_t at = (size_t)t * H + h;
-        decay[at] = expf(f + before - mine);
-        gain[at] = expf(i - mine);
+        decay[at] = expf(f[g] + before - mine);
+        gain[at] = expf(i[g] - mine);
         top_out[at] = mine;
       }
       top = __shfl_sync(0xffffffffu, mine, 31);  // (lanes past the end carry the last real maximum)
     }
-    if (lane == 0) *ts = top;
   }
+  if (lane == 0) *ts = top;
 }
 
 template <typename T>
@@ -367,8 +378,8 @@ extern "C" int asb_capped_gates_scan(float* decay, float* gain, float* top_out, 
                                      cudaStream_t stream) {
   if (R == 0) return 0;
   if (H < 1 || !(cap > 0.f)) return asb::fail("capped_gates_scan: %d heads, cap %f", H, cap);
-  const int threads = 32 * (H < 16 ? H : 16);
-  asb::launch(capped_gates_scan_kernel, R, threads, 0, stream, decay, gain, top_out, z, z_stride, i_off, f_off, i_bias,
+  if (H > 65535) return asb::fail("capped_gates_scan: %d heads exceed the grid", H);
+  asb::launch(capped_gates_scan_kernel, dim3(R, H), 32, 0, stream, decay, gain, top_out, z, z_stride, i_off, f_off, i_bias,
               f_bias, top_state, state_slots, req_q_start, H, cap);
   return asb::check_launch("capped_gates_scan");
 }

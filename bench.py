@@ -1277,7 +1277,7 @@ def time_vilulix(widths: list[int], layers: int, steps: int, warmup: int, pk: di
         KV, window = max(H // 4, 1), 1024
         pages_per = ctx // bs
         tables, t1 = i32([[r * pages_per + j for j in range(pages_per)] for r in range(B)]), i32([list(range(pages_per))])
-        starts, at = i32(list(range(B + 1))), i32([ctx - 1] * B)
+        starts, at, whole, first = i32(list(range(B + 1))), i32([ctx - 1] * B), i32([0, T]), i32([0])
         k_pages = torch.randn(B * pages_per, KV, bs, hd, device="cuda", dtype=bf)
         v_pages = torch.randn_like(k_pages)
         sink = torch.zeros(H, device="cuda")
@@ -1287,7 +1287,7 @@ def time_vilulix(widths: list[int], layers: int, steps: int, warmup: int, pk: di
             ms = timed(lambda: ops.paged_attention(q, k_pages, v_pages, tables, starts, at, num_requests=B, max_context=ctx, window=window,
                                                    scale=0.088, host_q_lens=[1] * B, sink=sk))  # fmt: skip
             kern[f"{name}_decode_b64"] = {"ms": round(ms, 4), "hbm_frac": round(2.0 * B * window * KV * hd * 2 / (ms * 1e-3) / bw, 3)}
-            ms = timed(lambda: ops.paged_attention(qp, k_pages, v_pages, t1, i32([0, T]), i32([0]), num_requests=1, max_context=T,
+            ms = timed(lambda: ops.paged_attention(qp, k_pages, v_pages, t1, whole, first, num_requests=1, max_context=T,
                                                    window=window, scale=0.088, host_q_lens=[T], sink=sk), 4)  # fmt: skip
             kern[f"{name}_prefill"] = {"ms": round(ms, 3), "tc_frac": round(4.0 * seen * H * hd / (ms * 1e-3) / tf, 4)}
         # between projection and attention: norm over the projection, rotation, page write, beside the norm per head
@@ -1312,7 +1312,7 @@ def time_vilulix(widths: list[int], layers: int, steps: int, warmup: int, pk: di
         for name, rows in (("prefill", T), ("decode_b64", B)):
             q_lat = torch.randn(rows, H, R + Rt, device="cuda")
             many = name == "prefill"
-            ms = timed(lambda: ops.latent_attention(q_lat, lat_pages, t1 if many else tables, i32([0, T]) if many else starts, i32([0]) if many else at,
+            ms = timed(lambda: ops.latent_attention(q_lat, lat_pages, t1 if many else tables, whole if many else starts, first if many else at,
                                                     rank=R, num_requests=1 if many else B, max_context=ctx, scale=0.07), 4)  # fmt: skip
             kern[f"latent_attention_{name}"] = {"ms": round(ms, 4), **({"tc_frac": round(2.0 * T * T / 2 * H * (2 * R + Rt) / (ms * 1e-3) / tf, 4)} if many else
                                                                       {"hbm_frac": round(B * ctx * (R + Rt) * 2 / (ms * 1e-3) / bw, 3)})}  # fmt: skip
